@@ -30,7 +30,7 @@
 extern "C" {
 #endif
 
-#define B200_ABI_VERSION 6
+#define B200_ABI_VERSION 7
 
 enum {
   B200_OK = 0,
@@ -388,6 +388,19 @@ int b200_frame_read_buffer(b200_frame* f, const char* name, void* dst_dev, int64
  *           g = exp(-exp(A_log[h]) softplus(W_a2 (W_a1 h) + dt_bias)), acting on the rows of S, and the gate
  *           sigmoid(W_g2 (W_g1 h)) on the normed result; portions of at least 16 tokens run in chunks of 32, the rest token by token
  *   mlp     B200_MLP_DENSE_RELU2 on its own norm
+ * and (the Megolorn design):
+ *   block   B200_BLOCK_PARALLEL_RESIDUAL with norm B200_NORM_LAYER: a layer norm with a weight and no bias instead of the RMS norm
+ *   mixer   B200_MIXER_DIFF_ATTENTION: every head has two query / key maps of size dim (rows laid out head by head as [map 1, map 2])
+ *           over the same values; q and k take a bias (bias), an RMS norm per head and map with one weight row (qk_norm) and rotary
+ *           positions (rot_scaling B200_ROT_LINEAR: every frequency divided by rot_factor); position p attends to the keys of its own
+ *           chunk of `chunk` positions up to itself (chunk = 0: all up to itself); o = a1 - lambda a2 with lambda =
+ *           exp(lq1.lk1) - exp(lq2.lk2) + diff, divided by its root mean square over the head's values, times (1 - diff), times
+ *           sigmoid((W_g h)_head) (head_gate); kv_from = j >= 0: the layer has no keys and values and reads layer j's cache
+ *   mlp     B200_MLP_DENSE_CLAMPED_GLU: W_down (g * sigmoid(1.702 g) * (u + 1)) with g and u bounded by expert_limit as above
+ *           B200_MLP_MOE_SILU_GLU: routed experts W_down (silu(W_gate h) * (W_up h)); fp32 scores = softmax over all experts + identity
+ *           router outputs; the choice adds a correction and, with groups > 1, is limited to the groups_keep groups of neighbouring
+ *           outputs with the largest single choice score; the `top` best are used with their plain scores as weights; the last
+ *           `identity` outputs are experts that return h itself; shared_ff > 0: one more such expert runs for every token
  * Precision: compute_dtype B200_BF16 = bf16 weights / activations / cache with fp32 accumulation, while norms, attention
  * scores and weights, gates, routers, recurrent state, the residual stream and the depth average stay fp32; B200_F32 =
  * everything in IEEE fp32 (FMA).
@@ -397,13 +410,16 @@ int b200_frame_read_buffer(b200_frame* f, const char* name, void* dst_dev, int64
 typedef struct b200_dlm b200_dlm;
 
 enum { B200_MIXER_LATENT_ATTENTION = 1, B200_MIXER_WINDOW_ATTENTION = 2, B200_MIXER_GLA = 3, B200_MIXER_MLSTM = 4, B200_MIXER_PARALLEL = 5,
-       B200_MIXER_SIGMOID_ATTENTION = 6, B200_MIXER_RETENTION = 7, B200_MIXER_DELTA = 8, B200_MIXER_MINGRU = 9, B200_MIXER_CHANNEL_DELTA = 10 };
-enum { B200_MLP_NONE = 0, B200_MLP_DENSE_RELU2 = 1, B200_MLP_MOE_RELU2 = 2, B200_MLP_DENSE_GATED_GELU = 3, B200_MLP_MOE_CLAMPED_GLU = 4 };
+       B200_MIXER_SIGMOID_ATTENTION = 6, B200_MIXER_RETENTION = 7, B200_MIXER_DELTA = 8, B200_MIXER_MINGRU = 9, B200_MIXER_CHANNEL_DELTA = 10,
+       B200_MIXER_DIFF_ATTENTION = 11 };
+enum { B200_MLP_NONE = 0, B200_MLP_DENSE_RELU2 = 1, B200_MLP_MOE_RELU2 = 2, B200_MLP_DENSE_GATED_GELU = 3, B200_MLP_MOE_CLAMPED_GLU = 4,
+       B200_MLP_DENSE_CLAMPED_GLU = 5, B200_MLP_MOE_SILU_GLU = 6 };
+enum { B200_NORM_RMS_ZERO_CENTRED = 0, B200_NORM_LAYER = 1 };   /* norm of the parallel-residual block */
 enum { B200_BLOCK_GATED_DEPTH_AVERAGE = 0, B200_BLOCK_SANDWICH = 1, B200_BLOCK_PARALLEL_RESIDUAL = 2, B200_BLOCK_PRE_NORM_STREAMS = 3 };
 enum { B200_SINK_LEARNED = 0, B200_SINK_NONE = 1, B200_SINK_UNIT = 2 };   /* what a softmax denominator holds beside the keys */
 #define B200_DLM_MAX_STREAMS 8
 enum { B200_ROT_HALVES = 0, B200_ROT_ADJACENT = 1 };          /* rot_pairing: dimension i with i + rot_dims / 2, or 2i with 2i + 1 */
-enum { B200_ROT_PLAIN = 0, B200_ROT_BANDS = 1, B200_ROT_RAMP = 2 };   /* rot_scaling */
+enum { B200_ROT_PLAIN = 0, B200_ROT_BANDS = 1, B200_ROT_RAMP = 2, B200_ROT_LINEAR = 3 };   /* rot_scaling */
 #define B200_DLM_MAX_DECAY_HEADS 256
 
 typedef struct {
@@ -420,14 +436,19 @@ typedef struct {
   float tau;                  /* GLA: decay = sigmoid(z)^(1 / tau)                              */
   int rot_pairing;            /* B200_ROT_HALVES / B200_ROT_ADJACENT                            */
   int rot_scaling;            /* B200_ROT_PLAIN; BANDS: rot_factor, rot_low, rot_high, rot_original (wavelength bands);
-                                 RAMP: rot_factor, rot_original, rot_fast, rot_slow (turns over rot_original positions at which the ramp starts / ends) */
+                                 RAMP: rot_factor, rot_original, rot_fast, rot_slow (turns over rot_original positions at which the ramp starts / ends);
+                                 LINEAR: rot_factor */
   float rot_fast, rot_slow;
   float softcap;              /* sigmoid attention: cap of the scaled score (<= 0: none)        */
   int v_mix;                  /* sigmoid attention: values blended with the first v_mix layer's */
   const float* decay;         /* retention: [heads] decays (copied by create)                   */
   int bias;                   /* the q / k / v (minGRU: z / x) projections add a bias           */
   int sink;                   /* B200_SINK_*                                                    */
-  int head_gate;              /* latent attention: a sigmoid gate per head on the result        */
+  int head_gate;              /* latent / differential attention: a sigmoid gate per head on the result */
+  int chunk;                  /* differential attention: keys of the query's own chunk of this many positions (0: all earlier ones) */
+  int qk_norm;                /* differential attention: RMS norm per head and map on q and k   */
+  float diff;                 /* differential attention: lambda's constant; the result is scaled by 1 - diff */
+  int kv_from;                /* differential attention: layer whose cached keys and values are read (-1: the layer's own) */
 } b200_dlm_mixer;
 
 typedef struct {
@@ -436,9 +457,12 @@ typedef struct {
   int mlp;                    /* B200_MLP_*                                                     */
   int ff;                     /* hidden size of the feed-forward (of one expert)                */
   int experts, top;           /* routed experts and how many of them a token uses               */
-  float expert_limit;         /* clamped experts: bound of the gate (above) and of the value (both sides) */
+  float expert_limit;         /* clamped gated units (experts or dense): bound of the gate (above) and of the value (both sides) */
   float router_scale;         /* clamped experts: multiplies the normalised weights             */
   float a_scale, b_scale;     /* pre-norm streams, PARALLEL: the pair's results are summed with these factors */
+  int shared_ff;              /* MOE_SILU_GLU: hidden size of the expert that runs for every token (0: none) */
+  int identity;               /* MOE_SILU_GLU: router outputs behind the experts that stand for h itself */
+  int groups, groups_keep;    /* MOE_SILU_GLU: equal groups of router outputs, and how many of them a token may choose from (groups <= 1: no limit) */
 } b200_dlm_layer;
 
 typedef struct {
@@ -452,6 +476,7 @@ typedef struct {
   int streams;                /* pre-norm streams: residual streams (0: one plain residual, no read / write weights) */
   float logit_scale;          /* pre-norm streams: multiplies the logits                         */
   int tied_head;              /* the logits come from the embedding table (no "head" tensor)     */
+  int norm;                   /* parallel residual: B200_NORM_*                                  */
 } b200_dlm_config;
 
 int b200_dlm_create(const b200_dlm_config* cfg, b200_dlm** out);

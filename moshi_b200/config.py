@@ -270,15 +270,18 @@ def tiny_lm_config(**over) -> LMConfig:
 # Decoder LMs given as a list of layers (text-only; no reference counterpart)
 # ---------------------------------------------------------------------------------------------------
 MIXERS = {"latent_attention": 1, "window_attention": 2, "gla": 3, "mlstm": 4, "parallel": 5,    # name -> B200_MIXER_*
-          "sigmoid_attention": 6, "retention": 7, "delta": 8, "mingru": 9, "channel_delta": 10}
+          "sigmoid_attention": 6, "retention": 7, "delta": 8, "mingru": 9, "channel_delta": 10,
+          "diff_attention": 11}
 # feed-forward kind -> B200_MLP_*: "dense" / "moe" are the squared-ReLU layers (a null "mlp" = none), "gated_gelu" a gated dense
-# layer with the tanh form of GELU, "moe_clamped_glu" routed experts with clamped gates behind a sigmoid router
-MLP_KINDS = {None: 0, "dense": 1, "moe": 2, "gated_gelu": 3, "moe_clamped_glu": 4}
+# layer with the tanh form of GELU, "moe_clamped_glu" routed experts with clamped gates behind a sigmoid router, "clamped_glu" such
+# a gated unit alone, "moe_silu_glu" routed experts with silu gates behind a softmax router (groups, identity and shared experts)
+MLP_KINDS = {None: 0, "dense": 1, "moe": 2, "gated_gelu": 3, "moe_clamped_glu": 4, "clamped_glu": 5, "moe_silu_glu": 6}
 BLOCKS = {"gated_depth_average": 0, "sandwich": 1, "parallel_residual": 2, "pre_norm_streams": 3}  # block arrangement -> B200_BLOCK_*
 NO_WINDOW = 1 << 30                                                                               # a window attention without a mask: every earlier key is seen
 SINKS = {"learned": 0, "none": 1, "unit": 2}                                                      # softmax denominator's extra term -> B200_SINK_*
 ROT_PAIRINGS = {"halves": 0, "adjacent": 1}                                                       # -> B200_ROT_HALVES / B200_ROT_ADJACENT
-ROT_SCALINGS = {None: 0, "bands": 1, "ramp": 2}                                                   # -> B200_ROT_PLAIN / BANDS / RAMP
+ROT_SCALINGS = {None: 0, "bands": 1, "ramp": 2, "linear": 3}                                      # -> B200_ROT_PLAIN / BANDS / RAMP / LINEAR
+NORMS = {"rms_zero_centred": 0, "layer": 1}                                                       # norm of the parallel-residual block -> B200_NORM_*
 
 
 @dataclass
@@ -299,7 +302,10 @@ class MixerConfig:
     recurrence of ``dim`` channels.  ``bias``: the q / k / v (or gate / candidate) projections add a bias.  ``sink``: what the
     softmax denominator holds beside the keys ("learned": exp of a weight per head, "none", "unit": one).  ``head_gate``: a
     sigmoid gate per head on the attention's result.  A ``latent_attention`` with ``rot_dims`` > 0 has that many rotated
-    query / key dimensions per head beside its ``dim`` unrotated ones; the rotated key part is one row shared by the heads."""
+    query / key dimensions per head beside its ``dim`` unrotated ones; the rotated key part is one row shared by the heads.
+    ``diff_attention``: two query / key maps per head over the same values, combined as a1 - lambda a2 (``diff`` is lambda's
+    constant), keys of the query's own ``chunk`` of positions (0: all earlier ones), ``qk_norm`` an RMS norm per head and map,
+    ``kv_from`` the layer whose cached keys and values are read (-1: its own); ``rot_scaling_kind`` "linear" reads {factor}."""
     kind: str
     heads: int
     dim: int
@@ -324,6 +330,10 @@ class MixerConfig:
     sink: str = "learned"
     head_gate: bool = False
     gate_rank: int = 16
+    chunk: int = 0
+    qk_norm: bool = False
+    diff: float = 0.0
+    kv_from: int = -1
 
 
 def _window_attention_from_dict(m: dict) -> MixerConfig:
@@ -361,6 +371,10 @@ class DecoderLayerConfig:
     router_scale: float = 1.0
     a_scale: float = 1.0                # a parallel pair whose results are summed with constant factors
     b_scale: float = 1.0
+    shared_ff: int = 0                  # moe_silu_glu: hidden size of the expert that runs for every token
+    identity: int = 0                   # router outputs behind the experts that stand for the input itself
+    groups: int = 1                     # equal groups of router outputs; a token chooses from the best ``groups_keep`` of them
+    groups_keep: int = 1
 
     @staticmethod
     def from_dict(d: dict) -> "DecoderLayerConfig":
@@ -431,6 +445,7 @@ class DecoderLMConfig:
     streams: int = 0                    # pre_norm_streams: residual streams with learned read / write weights (0: one plain residual)
     logit_scale: float = 1.0
     tied_head: bool = False             # the logits come from the embedding table
+    norm: str = "rms_zero_centred"      # parallel_residual: the block's norm
 
     @staticmethod
     def from_dict(d: dict) -> "DecoderLMConfig":
@@ -753,5 +768,103 @@ class DibulixConfig(DecoderLMConfig):
         return out
 
 
+@dataclass
+class MegolornConfig(DecoderLMConfig):
+    """``config.json`` of the Megolorn design: parallel blocks (one layer norm without bias feeds mixer and feed-forward,
+    ``x += mixer(h) + ff(h)``), a scaled embedding, layers of type ``attention`` (differential softmax attention on the query's own
+    chunk of positions, biased projections, a norm per head and map on queries and keys, rotation of adjacent pairs with linear
+    scaling, a gate per head; ``kv_from`` reads an earlier layer's keys and values), each with a ``dense`` (bounded gated unit) or
+    ``moe`` (softmax router with a choice correction, groups, identity experts and a shared expert) feed-forward or none."""
+
+    @staticmethod
+    def _layer(i: int, d: dict) -> DecoderLayerConfig:
+        t, m, mlp = d["type"], d["mixer"], d.get("mlp")
+        if t != "attention":
+            raise ValueError(f"layer {i}: a Megolorn layer is of type 'attention', not {t!r}")
+        rot = _rot_fields(m, "adjacent")
+        if rot["rot_scaling"]:
+            rot["rot_scaling_kind"] = "linear"
+        src = m.get("kv_from")
+        a = MixerConfig(kind="diff_attention", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                        scale=float(m["scale"]), chunk=int((m.get("mask") or {}).get("size") or 0), qk_norm=True, bias=True, sink="none",
+                        head_gate=True, diff=float(m["diff"]), kv_from=-1 if src is None else int(src), **rot)
+        kw: dict = dict(type="diff_attention", a=a)
+        if mlp is None:
+            return DecoderLayerConfig(mlp_kind=None, **kw)
+        if mlp["kind"] == "dense":
+            return DecoderLayerConfig(mlp_kind="clamped_glu", ff=int(mlp["ff"]), expert_limit=float(mlp["limit"]), **kw)
+        if mlp["kind"] != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        r, g, sh = mlp["router"], mlp["router"].get("groups") or {}, mlp.get("shared") or {}
+        return DecoderLayerConfig(mlp_kind="moe_silu_glu", ff=int(mlp["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]),
+                                  identity=int(r.get("identity") or 0), groups=int(g.get("count", 1)), groups_keep=int(g.get("keep", 1)),
+                                  shared_ff=int(sh.get("ff", 0)), **kw)
+
+    @staticmethod
+    def from_dict(d: dict) -> "MegolornConfig":
+        layers = [MegolornConfig._layer(i, x) for i, x in enumerate(d["layers"])]
+        for i, L in enumerate(layers):
+            j = L.a.kv_from
+            if j >= 0 and (j >= i or layers[j].a.kv_from >= 0 or
+                           any(getattr(layers[j].a, k) != getattr(L.a, k) for k in ("heads", "kv_heads", "dim", "vdim"))):
+                raise ValueError(f"layer {i}: kv_from = {j} must name an earlier layer with keys and values of its own and equal head counts and sizes")
+        return MegolornConfig(architecture=d["architecture"], vocab=int(d["vocab"]), width=int(d["width"]), layers=layers,
+                              embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)), norm_eps=float(d["norm"]["eps"]),
+                              block="parallel_residual", norm="layer")
+
+    @staticmethod
+    def _layer_to_dict(L: DecoderLayerConfig) -> dict:
+        a = L.a
+        mixer: dict = {"diff": a.diff, "dim": a.dim, "heads": a.heads, "kv_heads": a.kv_heads, "scale": a.scale, "vdim": a.vdim}
+        if a.kv_from >= 0:
+            mixer["kv_from"] = a.kv_from
+        if a.chunk:
+            mixer["mask"] = {"size": a.chunk}
+        rot = _rot_to_dict(a)
+        if rot is not None:
+            mixer["rot"] = rot
+        if L.mlp_kind is None:
+            mlp = None
+        elif L.mlp_kind == "clamped_glu":
+            mlp = {"ff": L.ff, "kind": "dense", "limit": L.expert_limit}
+        else:
+            router: dict = {"experts": L.experts, "identity": L.identity, "top": L.top}
+            if L.groups > 1:
+                router["groups"] = {"count": L.groups, "keep": L.groups_keep}
+            mlp = {"expert": {"ff": L.ff}, "kind": "moe", "router": router}
+            if L.shared_ff:
+                mlp["shared"] = {"ff": L.shared_ff}
+        return {"mixer": mixer, "mlp": mlp, "type": "attention"}
+
+    def to_dict(self) -> dict:
+        return {"architecture": self.architecture, "embedding": {"scale": self.embedding_scale},
+                "layers": [self._layer_to_dict(x) for x in self.layers], "norm": {"eps": self.norm_eps}, "vocab": self.vocab, "width": self.width}
+
+    def tensor_shapes(self) -> dict:
+        W = self.width
+        out = {"embed": (self.vocab, W)}
+        for i, L in enumerate(self.layers):
+            p, m, a = f"l{i}.", f"l{i}.mix.", L.a
+            out[p + "norm1"] = (W,)
+            own = a.kv_from < 0
+            for nm, rows in (("q", 2 * a.heads * a.dim),) + ((("k", 2 * a.kv_heads * a.dim), ("v", a.kv_heads * a.vdim)) if own else ()):
+                out.update({m + nm: (rows, W), m + nm + ".b": (rows,)})
+            out[m + "q.norm"] = (a.dim,)
+            if own:
+                out[m + "k.norm"] = (a.dim,)
+            out.update({m + nm: (a.dim,) for nm in ("lq1", "lk1", "lq2", "lk2")})
+            out.update({m + "g": (a.heads, W), m + "o": (W, a.heads * a.vdim)})
+            glu = [("mlp.", L.ff)] if L.mlp_kind == "clamped_glu" else []
+            if L.mlp_kind == "moe_silu_glu":
+                n = L.experts + L.identity
+                glu = [(f"mlp.e{e}.", L.ff) for e in range(L.experts)] + ([("mlp.shared.", L.shared_ff)] if L.shared_ff else [])
+                out.update({p + "mlp.router": (n, W), p + "mlp.correction": (n,)})
+            for q, F in glu:
+                out.update({p + q + "gate": (F, W), p + q + "up": (F, W), p + q + "down": (W, F)})
+        out.update({"final.norm": (W,), "head": (self.vocab, W)})
+        return out
+
+
 # architecture name in config.json -> configuration class (the model registry of the text-only decoder LMs)
-DECODER_ARCHITECTURES: dict = {"Likosun": DecoderLMConfig, "Govuvik": GovuvikConfig, "Namalix": NamalixConfig, "Dibulix": DibulixConfig}
+DECODER_ARCHITECTURES: dict = {"Likosun": DecoderLMConfig, "Govuvik": GovuvikConfig, "Namalix": NamalixConfig, "Dibulix": DibulixConfig,
+                               "Megolorn": MegolornConfig}

@@ -1,9 +1,10 @@
 // Decoder-LM handle: a language model given as a list of layers (mixer + feed-forward per layer), its weights under the
 // checkpoint's names, a slot cache per layer (latents, or keys and values, plus the carried inputs of convolutions and the
 // state of recurrent mixers), and the ragged step (any number of new tokens per slot) that both prompt portions and
-// single-token decoding go through.  Two block arrangements are registered: gated parallel sublayers with a depth-weighted
-// average (the Likosun design), RMS-norm sandwiches around mixer and feed-forward in turn (the Govuvik design), and a plain
-// parallel block on one zero-centred RMS norm (the Namalix design).
+// single-token decoding go through.  Block arrangements: gated parallel sublayers with a depth-weighted
+// average (the Likosun design), RMS-norm sandwiches around mixer and feed-forward in turn (the Govuvik design), a plain parallel
+// block on one zero-centred RMS norm (the Namalix design) or one layer norm (the Megolorn design), and pre-norm sublayers on
+// residual streams (the Dibulix design).
 #include <algorithm>
 
 #include <cmath>
@@ -12,6 +13,7 @@
 #include "dlm_mixers.cuh"
 #include "dlm_mixers2.cuh"
 #include "dlm_mixers3.cuh"
+#include "dlm_mixers4.cuh"
 #include "gemm_sk.cuh"
 #include "lm_kernels.cuh"
 
@@ -72,6 +74,11 @@ struct Layer {
   int g_z = 0, g_x = 0, g_g = 0, c_a1 = 0, c_g1 = 0, gate_rank = 0;
   float *qkv_bias = nullptr, *zx_bias = nullptr, *gru = nullptr;      // gru: [slots][channels] state of the minGRU
   void* g2 = nullptr;                  // T [heads * vdim][gate_rank]
+  // ---- differential attention on the parallel-residual block: projection [q | k | v | gate | up] (no k, v with kv_from; gate and up of
+  // a dense or shared gated unit), output product [o | down] on rows [heads' results | gated unit] of ob_ld elements
+  int kv_src = -1, rot_id = -1, glu_ff = 0, ob_ld = 0, ob_act = 0, mma_vt = 0;
+  size_t smem_mma_one = 0;
+  float lambda = 0.f;
 };
 
 // attention tile list of one (heads, rows per tile) combination
@@ -136,6 +143,8 @@ struct b200_dlm {
   float* small32 = nullptr;            // [tokens][nsmall] fp32 results of the small projection
   float* xs = nullptr;                 // pre-norm streams block: the residual streams [tokens][streams][width]
   float *rows3 = nullptr, *gend = nullptr;      // chunked delta rule with a decay per key channel: [tokens][heads][3 dim], [chunks][heads][dim]
+  struct Rotation { b200_dlm_mixer m; double* freq; float* table; };
+  std::vector<Rotation> rots;          // distinct rotations of the differential attention layers; table: [tokens][rot_dims], filled once per step
   void *vfirst = nullptr, *act2 = nullptr;      // T [tokens][G * vdim] values of layer vmix_first; T [tokens * top][2 ff] experts' first product
 };
 
@@ -429,7 +438,9 @@ std::vector<double> rotary_frequencies(const b200_dlm_mixer& m) {
   const double two_pi = 6.283185307179586476925;
   for (int i = 0; i < half; ++i) {
     double v = std::pow((double)m.rot_base, -2.0 * i / m.rot_dims);
-    if (m.rot_factor > 0.f) {
+    if (m.rot_scaling == B200_ROT_LINEAR) {
+      v /= m.rot_factor;
+    } else if (m.rot_factor > 0.f) {
       const double wave = two_pi / v, orig = m.rot_original;
       if (wave < orig / m.rot_high) {
       } else if (wave > orig / m.rot_low) {
@@ -971,6 +982,160 @@ size_t sigmoid_attn_smem(const b200_dlm_mixer& m, int QT, int KT, size_t es, int
   return 4 * (QT * Nq + rows * m.vdim + 2 * rows * (KT + 1) + (size_t)m.heads * m.heads + m.heads) + es * ((size_t)KT * *kstride + KT * Nv) + 32;
 }
 
+// the gated experts of a layer: rows 2f / 2f + 1 of an expert's first matrix are gate f / value f
+int put_glu_experts(b200_dlm* h, Layer& L, const std::string& p) {
+  const int64_t W = h->cfg.width, E = L.c.experts, F = L.c.ff;
+  const size_t es = esize(h);
+  B200_TRY(h->weights.alloc(&L.ups, (size_t)E * 2 * F * W * es, false));
+  B200_TRY(h->weights.alloc(&L.downs, (size_t)E * W * F * es, false));
+  void *tg = nullptr, *tu = nullptr;
+  B200_CUDA(cudaMalloc(&tg, (size_t)F * W * es));
+  B200_CUDA(cudaMalloc(&tu, (size_t)F * W * es));
+  int rc = B200_OK;
+  for (int64_t e = 0; e < E && rc == B200_OK; ++e) {
+    const std::string q = p + "mlp.e" + std::to_string(e) + ".";
+    rc = put_matrix(h, q + "gate", F, W, tg);
+    if (rc == B200_OK) rc = put_matrix(h, q + "up", F, W, tu);
+    if (rc != B200_OK) break;
+    char* dst = static_cast<char*>(L.ups) + (size_t)e * 2 * F * W * es;
+    const unsigned g = (unsigned)ceil_div64(F * W, 256);
+    if (h->f32) interleave_rows_kernel<float><<<g, 256>>>(static_cast<const float*>(tg), static_cast<const float*>(tu), reinterpret_cast<float*>(dst), F, W);
+    else interleave_rows_kernel<bf16><<<g, 256>>>(static_cast<const bf16*>(tg), static_cast<const bf16*>(tu), reinterpret_cast<bf16*>(dst), F, W);
+    rc = check_launch("interleave_rows");
+    if (rc == B200_OK) rc = put_matrix(h, q + "down", W, F, static_cast<char*>(L.downs) + (size_t)e * W * F * es);
+  }
+  cudaDeviceSynchronize();
+  cudaFree(tg); cudaFree(tu);
+  B200_TRY(rc);
+  h->weight_bytes += 3 * E * F * W * es;
+  return B200_OK;
+}
+
+// a layer of the parallel-residual block with differential attention (its norm is loaded already)
+int finalize_diff_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
+  Layer& L = h->layers[i];
+  const b200_dlm_mixer& a = L.c.a;
+  const int64_t W = h->cfg.width;
+  const size_t es = esize(h);
+  const std::string p = "l" + std::to_string(i) + ".", m = p + "mix.";
+  const int H = a.heads, G = a.kv_heads;
+  const bool own = a.kv_from < 0, dense = L.c.mlp == B200_MLP_DENSE_CLAMPED_GLU, moe = L.c.mlp == B200_MLP_MOE_SILU_GLU;
+  auto pad8 = [](int v) { return (v + 7) / 8 * 8; };
+  L.kv_src = own ? i : a.kv_from;
+  L.Nq = 2 * H * a.dim; L.Nk = 2 * G * a.dim; L.Nv = G * a.vdim;
+  L.glu_ff = dense ? L.c.ff : moe ? L.c.shared_ff : 0;
+  const std::string glu = p + (dense ? "mlp." : "mlp.shared.");
+  L.p_q = 0; L.p_k = L.Nq; L.p_v = L.p_k + (own ? L.Nk : 0); L.p_ffg = pad8(L.p_v + (own ? L.Nv : 0)); L.p_ffu = pad8(L.p_ffg + L.glu_ff);
+  L.ncat = L.glu_ff ? L.p_ffu + L.glu_ff : L.p_v + (own ? L.Nv : 0);
+  L.ldp = pad8(L.ncat);
+  void* cat = nullptr;
+  B200_TRY(h->weights.alloc(&cat, (size_t)L.ncat * W * es, true));
+  auto at = [&](int off) { return static_cast<char*>(cat) + (size_t)off * W * es; };
+  B200_TRY(put_matrix(h, m + "q", L.Nq, W, at(L.p_q)));
+  if (own) {
+    B200_TRY(put_matrix(h, m + "k", L.Nk, W, at(L.p_k)));
+    B200_TRY(put_matrix(h, m + "v", L.Nv, W, at(L.p_v)));
+  }
+  if (L.glu_ff) {
+    B200_TRY(put_matrix(h, glu + "gate", L.glu_ff, W, at(L.p_ffg)));
+    B200_TRY(put_matrix(h, glu + "up", L.glu_ff, W, at(L.p_ffu)));
+  }
+  B200_TRY(seal_weight(h, L.cat, cat, L.ncat, (int)W, drop));
+  if (a.bias) {
+    const int C = L.Nq + (own ? L.Nk + L.Nv : 0);
+    B200_TRY(h->weights.alloc_t(&L.qkv_bias, (size_t)C, false));
+    const Tensor* t = nullptr;
+    int off = 0;
+    for (const char* nm : {"q", "k", "v"}) {
+      if (!own && nm[0] != 'q') break;
+      const int rows = nm[0] == 'q' ? L.Nq : nm[0] == 'k' ? L.Nk : L.Nv;
+      B200_TRY(find_tensor(h, m + nm + ".b", {rows}, &t));
+      B200_TRY(convert_into(t, L.qkv_bias + off));
+      off += rows;
+    }
+    h->weight_bytes += (int64_t)C * 4;
+  }
+  if (a.qk_norm) {
+    B200_TRY(get_f32(h, m + "q.norm", a.dim, &L.qnorm));
+    if (own) B200_TRY(get_f32(h, m + "k.norm", a.dim, &L.knorm));
+  }
+  {   // lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff
+    double dot[2];
+    std::vector<float> u(a.dim), v(a.dim);
+    for (int k = 0; k < 2; ++k) {
+      float *du = nullptr, *dv = nullptr;
+      B200_TRY(get_f32(h, m + "lq" + std::to_string(k + 1), a.dim, &du));
+      B200_TRY(get_f32(h, m + "lk" + std::to_string(k + 1), a.dim, &dv));
+      B200_CUDA(cudaMemcpy(u.data(), du, (size_t)a.dim * 4, cudaMemcpyDeviceToHost));
+      B200_CUDA(cudaMemcpy(v.data(), dv, (size_t)a.dim * 4, cudaMemcpyDeviceToHost));
+      dot[k] = 0.0;
+      for (int d = 0; d < a.dim; ++d) dot[k] += (double)u[d] * v[d];
+    }
+    L.lambda = (float)(std::exp(dot[0]) - std::exp(dot[1]) + a.diff);
+  }
+  if (a.rot_dims > 0) {      // layers with the same rotation share its table
+    for (size_t k = 0; k < h->rots.size() && L.rot_id < 0; ++k) {
+      const b200_dlm_mixer& r = h->rots[k].m;
+      if (r.rot_dims == a.rot_dims && r.rot_base == a.rot_base && r.rot_scaling == a.rot_scaling && r.rot_factor == a.rot_factor) L.rot_id = (int)k;
+    }
+    if (L.rot_id < 0) {
+      b200_dlm::Rotation r{a, nullptr, nullptr};
+      const std::vector<double> fr = rotary_frequencies(a);
+      B200_TRY(h->weights.alloc_t(&r.freq, fr.size(), false));
+      B200_CUDA(cudaMemcpy(r.freq, fr.data(), fr.size() * sizeof(double), cudaMemcpyHostToDevice));
+      h->rots.push_back(r);
+      L.rot_id = (int)h->rots.size() - 1;
+    }
+  }
+  // the small fp32 projection: head gates | router logits
+  const int n_route = moe ? L.c.experts + L.c.identity : 0;
+  L.s_gate = 0; L.s_router = a.head_gate ? H : 0; L.nsmall = L.s_router + n_route;
+  if (L.nsmall) {
+    B200_TRY(h->weights.alloc(&L.w_small, (size_t)L.nsmall * W * es, false));
+    auto sat = [&](int off) { return static_cast<char*>(L.w_small) + (size_t)off * W * es; };
+    if (a.head_gate) B200_TRY(put_matrix(h, m + "g", H, W, sat(L.s_gate)));
+    if (moe) B200_TRY(put_matrix(h, p + "mlp.router", n_route, W, sat(L.s_router)));
+    h->weight_bytes += (int64_t)L.nsmall * W * es;
+  }
+  // both sublayers' output products as one: [o | down] against rows [heads' results | gated unit]
+  const int Kv = H * a.vdim;
+  L.ob_act = pad8(Kv); L.ob_ld = L.glu_ff ? pad8(L.ob_act + L.glu_ff) : Kv;
+  void *wo = nullptr, *tmp = nullptr;
+  B200_TRY(h->weights.alloc(&wo, (size_t)W * L.ob_ld * es, true));
+  B200_CUDA(cudaMalloc(&tmp, (size_t)W * std::max(Kv, L.glu_ff) * es));
+  int rc = put_matrix(h, m + "o", W, Kv, tmp);
+  if (rc == B200_OK && cudaMemcpy2D(wo, (size_t)L.ob_ld * es, tmp, (size_t)Kv * es, (size_t)Kv * es, (size_t)W, cudaMemcpyDeviceToDevice) != cudaSuccess) rc = B200_ERR_CUDA;
+  if (rc == B200_OK && L.glu_ff) {
+    rc = put_matrix(h, glu + "down", W, L.glu_ff, tmp);
+    if (rc == B200_OK && cudaMemcpy2D(static_cast<char*>(wo) + (size_t)L.ob_act * es, (size_t)L.ob_ld * es, tmp, (size_t)L.glu_ff * es, (size_t)L.glu_ff * es, (size_t)W, cudaMemcpyDeviceToDevice) != cudaSuccess) rc = B200_ERR_CUDA;
+  }
+  cudaDeviceSynchronize();
+  cudaFree(tmp);
+  B200_TRY(rc);
+  B200_TRY(seal_weight(h, L.o, wo, (int)W, L.ob_ld, drop, (int)W));
+  if (moe) {
+    B200_TRY(get_f32(h, p + "mlp.correction", n_route, &L.correction));
+    B200_TRY(put_glu_experts(h, L, p));
+  }
+  // kernels: rows are (token, query head of one key/value head)
+  const int rep = H / G;
+  L.QT = 0;
+  for (int kt : {32, 16, 8})
+    for (int mr : {8, 4, 1}) {
+      const size_t sm = diff_attn_smem(a.dim, a.vdim, mr, kt);
+      if (!L.QT && sm <= 200 * 1024) { L.QT = mr; L.KT = kt; L.attn_smem = sm; }
+    }
+  if (!L.QT) B200_FAIL(B200_ERR_SHAPE, "decoder LM: layer %d: the attention's heads do not fit shared memory", i);
+  L.sig = add_sig(h, rep, L.QT);
+  if (!h->f32 && a.dim % 16 == 0 && a.vdim % 16 == 0 && a.vdim <= 128) {
+    L.mma_vt = ceil_div(a.vdim, 32) * 2;
+    L.mma_smem = diff_attn_mma_smem(a.dim, L.mma_vt, false);
+    L.smem_mma_one = diff_attn_mma_smem(a.dim, L.mma_vt, true);
+    if (std::max(L.mma_smem, L.smem_mma_one) <= 220 * 1024) { L.sig_mma = add_sig(h, rep, 64); L.sig_one = add_sig(h, rep, 16); }
+  }
+  return B200_OK;
+}
+
 int finalize_parallel_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
   Layer& L = h->layers[i];
   const b200_dlm_config& c = h->cfg;
@@ -983,7 +1148,8 @@ int finalize_parallel_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
     return put_matrix(h, name, rows, K, *out);
   };
   B200_TRY(get_f32(h, p + "norm1", W, &L.n1w));
-  B200_LAUNCH(add_one_kernel, ceil_div((int)W, 256), 256, 0, nullptr, L.n1w, (int)W);
+  if (c.norm == B200_NORM_RMS_ZERO_CENTRED) B200_LAUNCH(add_one_kernel, ceil_div((int)W, 256), 256, 0, nullptr, L.n1w, (int)W);
+  if (L.c.mixer == B200_MIXER_DIFF_ATTENTION) return finalize_diff_layer(h, i, drop);
   const bool attn = L.c.mixer == B200_MIXER_SIGMOID_ATTENTION, ret = L.c.mixer == B200_MIXER_RETENTION, delta = L.c.mixer == B200_MIXER_DELTA;
   const int H = a.heads, G = attn || delta ? a.kv_heads : a.heads;
   L.Nq = (attn ? H : G) * a.dim; L.Nk = G * a.dim; L.Nv = (attn ? G : H) * a.vdim;
@@ -1089,28 +1255,7 @@ int finalize_parallel_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
     B200_TRY(seal_weight(h, L.down, wd, (int)W, F, drop, (int)W));
   } else if (moe) {
     B200_TRY(get_f32(h, p + "mlp.correction", E, &L.correction));
-    B200_TRY(h->weights.alloc(&L.ups, (size_t)E * 2 * F * W * es, false));      // rows 2f / 2f + 1 of an expert: gate f / value f
-    B200_TRY(h->weights.alloc(&L.downs, (size_t)E * W * F * es, false));
-    void *tg = nullptr, *tu = nullptr;
-    B200_CUDA(cudaMalloc(&tg, (size_t)F * W * es));
-    B200_CUDA(cudaMalloc(&tu, (size_t)F * W * es));
-    int rc = B200_OK;
-    for (int64_t e = 0; e < E && rc == B200_OK; ++e) {
-      const std::string q = p + "mlp.e" + std::to_string(e) + ".";
-      rc = put_matrix(h, q + "gate", F, W, tg);
-      if (rc == B200_OK) rc = put_matrix(h, q + "up", F, W, tu);
-      if (rc != B200_OK) break;
-      char* dst = static_cast<char*>(L.ups) + (size_t)e * 2 * F * W * es;
-      const unsigned g = (unsigned)ceil_div64((int64_t)F * W, 256);
-      if (h->f32) interleave_rows_kernel<float><<<g, 256>>>(static_cast<const float*>(tg), static_cast<const float*>(tu), reinterpret_cast<float*>(dst), F, W);
-      else interleave_rows_kernel<bf16><<<g, 256>>>(static_cast<const bf16*>(tg), static_cast<const bf16*>(tu), reinterpret_cast<bf16*>(dst), F, W);
-      rc = check_launch("interleave_rows");
-      if (rc == B200_OK) rc = put_matrix(h, q + "down", W, F, static_cast<char*>(L.downs) + (size_t)e * W * F * es);
-    }
-    cudaDeviceSynchronize();
-    cudaFree(tg); cudaFree(tu);
-    B200_TRY(rc);
-    h->weight_bytes += 3 * (int64_t)E * F * W * es;
+    B200_TRY(put_glu_experts(h, L, p));
   }
   return B200_OK;
 }
@@ -1170,13 +1315,107 @@ int sigmoid_attention(b200_dlm* h, const Layer& L, int n_tok, int max_ctx) {
   return B200_OK;
 }
 
-// routed experts with clamped gates on the rows of hb -> yexp [tokens * top][W]; the router's logits are in small32
+template <int VT, bool SK>
+int launch_diff_mma(cudaStream_t st, const DiffAttnParams& p, size_t smem) {
+  static bool attr_set = false;
+  if (!attr_set) {
+    B200_CUDA(cudaFuncSetAttribute((diff_attn_mma_kernel<VT, SK>), cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    attr_set = true;
+  }
+  B200_LAUNCH((diff_attn_mma_kernel<VT, SK>), dim3(p.n_tiles * p.G, p.nsplit), 128, smem, st, p);
+  return check_launch("diff_attn_mma");
+}
+
+template <bool SK>
+int launch_diff_mma_vt(cudaStream_t st, const DiffAttnParams& p, int vt, size_t smem) {
+  switch (vt) {
+    case 2: return launch_diff_mma<2, SK>(st, p, smem);
+    case 4: return launch_diff_mma<4, SK>(st, p, smem);
+    case 6: return launch_diff_mma<6, SK>(st, p, smem);
+    default: return launch_diff_mma<8, SK>(st, p, smem);
+  }
+}
+
+// which attention kernel a step takes: the tensor cores (16-row tiles whose warps share the keys when no request brings more rows), or the CUDA cores
+template <typename T>
+bool diff_attention_on_tensor_cores(const b200_dlm* h, const Layer& L) { return sizeof(T) == 2 && h->attn_tc && L.sig_mma >= 0; }
+
+// gate and up of the gated unit, queries, keys and values from the projection; then the attention -> obuf [tokens][ob_ld]
+template <typename T>
+int diff_attention(b200_dlm* h, const Layer& L, int n_tok, int max_ctx) {
+  const b200_dlm_mixer& a = L.c.a;
+  const Layer& S = h->layers[L.kv_src];
+  cudaStream_t st = h->stream;
+  const bool mma = diff_attention_on_tensor_cores<T>(h, L), own = a.kv_from < 0;
+  const int rep = a.heads / a.kv_heads;
+  {
+    DiffPrepParams p;
+    p.proj = h->proj; p.ld = L.ldp; p.off_q = L.p_q; p.off_k = own ? L.p_k : -1; p.off_v = L.p_v; p.Hm = 2 * a.heads; p.Gm = 2 * a.kv_heads; p.Nv = L.Nv;
+    p.dim = a.dim; p.half = a.rot_dims / 2; p.adjacent = a.rot_pairing == B200_ROT_ADJACENT; p.rot = L.rot_id >= 0 ? h->rots[L.rot_id].table : nullptr;
+    p.bias = L.qkv_bias; p.wq = L.qnorm; p.wk = L.knorm; p.eps = h->cfg.norm_eps; p.qscale = a.scale; p.qout = h->qkv32;
+    p.kcache = S.kcache; p.vcache = S.vcache; p.cap = h->cap; p.tok_slot = h->meta_dev + h->off_slot; p.tok_pos = h->meta_dev + h->off_pos;
+    p.off_g = L.p_ffg; p.off_u = L.p_ffu; p.F = L.glu_ff; p.glu = L.c.mlp == B200_MLP_DENSE_CLAMPED_GLU ? GLU_CLAMPED : GLU_SILU; p.limit = L.c.expert_limit;
+    p.act = static_cast<T*>(h->obuf) + L.ob_act; p.lda = L.ob_ld;
+    const dim3 grid(n_tok, 1 + ceil_div(L.glu_ff, GLU_SLICE));
+    const size_t smem = (size_t)8 * a.dim * sizeof(float);
+    TIMED(CLS_ELEMENTWISE, if (mma) B200_LAUNCH((diff_prep_kernel<T, bf16>), grid, 256, smem, st, p); else B200_LAUNCH((diff_prep_kernel<T, float>), grid, 256, smem, st, p));
+    B200_TRY(check_launch("diff_prep"));
+  }
+  const bool one = mma && h->max_entry_tokens * rep <= 16;
+  const TileSig& s = h->sigs[one ? L.sig_one : mma ? L.sig_mma : L.sig];
+  DiffAttnParams p;
+  p.q = h->qkv32; p.ldq = L.Nq; p.kcache = S.kcache; p.vcache = S.vcache;
+  p.tile_row0 = h->meta_dev + s.off_row0; p.tile_rows = h->meta_dev + s.off_rows; p.tile_slot = h->meta_dev + s.off_slot; p.tok_pos = h->meta_dev + h->off_pos;
+  p.gate = a.head_gate ? h->small32 + L.s_gate : nullptr; p.ldg = L.nsmall; p.out = h->obuf; p.ldo = L.ob_ld; p.part = h->part;
+  p.cap = h->cap; p.H = a.heads; p.G = a.kv_heads; p.dim = a.dim; p.vdim = a.vdim; p.chunk = a.chunk; p.n_tiles = s.count; p.MR = s.rpt; p.KT = mma ? DA_KT : L.KT;
+  p.lambda = L.lambda; p.out_scale = 1.f - a.diff; p.eps = h->cfg.norm_eps;
+  // keys are cut over several CTAs per tile when the tiles alone cannot fill the GPU (decoding, short portions)
+  const int seen = a.chunk > 0 ? std::min(max_ctx, a.chunk + s.rpt / rep) : max_ctx, key_tiles = ceil_div(seen, p.KT), ctas = s.count * a.kv_heads;
+  int nsplit = 1;
+  if (h->attn_split > 0) nsplit = std::min(h->attn_split, 64);
+  else if (ctas < 296) nsplit = std::min(296 / ctas, 64);
+  nsplit = a.vdim > 1024 ? 1 : std::max(1, std::min(nsplit, key_tiles));
+  while (nsplit > 1 && (size_t)ctas * nsplit * s.rpt * (2 * a.vdim + 4) > h->part_floats) --nsplit;
+  p.nsplit = nsplit;
+  B200_TRY(mark(h, CLS_ATTN));
+  if (mma) {
+    if constexpr (sizeof(T) == 2) B200_TRY(one ? launch_diff_mma_vt<true>(st, p, L.mma_vt, L.smem_mma_one) : launch_diff_mma_vt<false>(st, p, L.mma_vt, L.mma_smem));
+  } else {
+    static bool attr_set = false;
+    if (!attr_set) {
+      B200_CUDA(cudaFuncSetAttribute(diff_attn_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+      attr_set = true;
+    }
+    B200_LAUNCH(diff_attn_kernel<T>, dim3(ctas, nsplit), 256, L.attn_smem, st, p);
+    B200_TRY(check_launch("diff_attn"));
+  }
+  if (nsplit > 1) {
+    B200_LAUNCH(diff_attn_merge_kernel<T>, dim3(ctas, ceil_div(s.rpt, 4)), 128, 0, st, p);
+    B200_TRY(check_launch("diff_attn_merge"));
+  }
+  return mark(h, -1);
+}
+
+// routed gated experts on the rows of hb -> yexp [tokens * top][W]; the router's logits are in small32
 template <typename T>
 int routed_experts_glu(b200_dlm* h, const Layer& L, const T* hb, int n_tok) {
   const int W = h->cfg.width, E = L.c.experts, top = L.c.top, F = L.c.ff, pairs = n_tok * top;
+  const bool silu = L.c.mlp == B200_MLP_MOE_SILU_GLU;
   cudaStream_t st = h->stream;
-  B200_LAUNCH(moe_route_sigmoid_kernel, ceil_div(n_tok, 4), 128, 0, st, h->small32 + L.s_router, (long long)L.nsmall, L.correction, E, top, L.c.router_scale,
-              h->moe_idx, h->moe_w, n_tok);
+  if (silu) {
+    const int n = E + L.c.identity, groups = std::max(L.c.groups, 1);
+    const size_t smem = (size_t)4 * (2 * n + groups) * sizeof(float);
+    static bool attr_set = false;
+    if (!attr_set) {
+      B200_CUDA(cudaFuncSetAttribute(moe_route_softmax_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+      attr_set = true;
+    }
+    B200_LAUNCH(moe_route_softmax_kernel, ceil_div(n_tok, 4), 128, smem, st, h->small32 + L.s_router, (long long)L.nsmall, L.correction, n, top, groups, L.c.groups_keep,
+                h->moe_idx, h->moe_w, n_tok);
+  } else {
+    B200_LAUNCH(moe_route_sigmoid_kernel, ceil_div(n_tok, 4), 128, 0, st, h->small32 + L.s_router, (long long)L.nsmall, L.correction, E, top, L.c.router_scale,
+                h->moe_idx, h->moe_w, n_tok);
+  }
   bool mma = false;
   if constexpr (sizeof(T) == 2) mma = h->attn_tc && W % 16 == 0 && F % 16 == 0;
   const int tile_m = mma ? 128 : 64;
@@ -1199,14 +1438,14 @@ int routed_experts_glu(b200_dlm* h, const Layer& L, const T* hb, int n_tok) {
       }
       // gate and value rows of an expert are interleaved, so the first product's epilogue holds both of an output in one thread
       B200_LAUNCH(grouped_gemm_mma_kernel, dim3(ceil_div(2 * F, 128), max_tiles), 256, GG_SMEM, st, hb, (long long)W, h->moe_row_tok, ups, (long long)W, (long long)2 * F * W,
-                  act, (long long)F, (const int*)nullptr, h->moe_tile_e, h->moe_tile_r0, h->moe_tile_n, h->moe_ntiles, 2 * F, W, 2, L.c.expert_limit);
+                  act, (long long)F, (const int*)nullptr, h->moe_tile_e, h->moe_tile_r0, h->moe_tile_n, h->moe_ntiles, 2 * F, W, silu ? 3 : 2, L.c.expert_limit);
       B200_LAUNCH(grouped_gemm_mma_kernel, dim3(ceil_div(W, 128), max_tiles), 256, GG_SMEM, st, act, (long long)F, (const int*)nullptr, downs, (long long)F, (long long)W * F,
                   yexp, (long long)W, h->moe_perm, h->moe_tile_e, h->moe_tile_r0, h->moe_tile_n, h->moe_ntiles, W, F, 0, 0.f);
     }
   } else {
     B200_LAUNCH((grouped_gemm_kernel<T, T, T>), dim3(ceil_div(2 * F, 64), max_tiles), 256, 0, st, hb, (long long)W, h->moe_row_tok, ups, (long long)W, (long long)2 * F * W,
                 act2, (long long)2 * F, (const int*)nullptr, h->moe_tile_e, h->moe_tile_r0, h->moe_tile_n, h->moe_ntiles, 2 * F, W, 0);
-    B200_LAUNCH(clamped_glu_kernel<T>, (unsigned)ceil_div64(n, 256), 256, 0, st, act2, act, F, n, L.c.expert_limit);
+    B200_LAUNCH(interleaved_glu_kernel<T>, (unsigned)ceil_div64(n, 256), 256, 0, st, act2, act, F, n, L.c.expert_limit, silu ? 1 : 0);
     B200_LAUNCH((grouped_gemm_kernel<T, T, T>), dim3(ceil_div(W, 64), max_tiles), 256, 0, st, act, (long long)F, (const int*)nullptr, downs, (long long)F, (long long)W * F,
                 yexp, (long long)W, h->moe_perm, h->moe_tile_e, h->moe_tile_r0, h->moe_tile_n, h->moe_ntiles, W, F, 0);
   }
@@ -1286,15 +1525,25 @@ int step_parallel(b200_dlm* h, int n_tok, int n_want, int max_ctx, float* logits
   T* ob = static_cast<T*>(h->obuf);
   T* mixo = static_cast<T*>(h->mixo);
   TIMED(CLS_ELEMENTWISE, B200_LAUNCH(embed_scale_norm_kernel<T>, n_tok, 256, 0, st, meta + h->off_tok, static_cast<const T*>(h->embed), c.vocab, W, c.embedding_scale,
-                                     h->layers[0].n1w, h->xin, hb, c.norm_eps, h->err));
+                                     h->layers[0].n1w, h->xin, hb, c.norm_eps, h->err, c.norm == B200_NORM_LAYER));
+  for (const auto& r : h->rots)
+    TIMED(CLS_ELEMENTWISE, B200_LAUNCH(rotary_table_kernel, n_tok, 64, 0, st, tok_pos, r.freq, r.m.rot_dims / 2, 1.f, r.table));
   for (int li = 0; li < c.n_layers; ++li) {
     const Layer& L = h->layers[li];
     const b200_dlm_mixer& a = L.c.a;
     const bool last = li + 1 == c.n_layers;
     TIMED(CLS_LINEAR, B200_TRY(linear<T>(h, hb, W, L.cat, proj, L.ldp, n_tok)));
-    if (L.nsmall) TIMED(CLS_FOLD, B200_TRY(small_proj<T>(h, hb, W, L.w_small, nullptr, h->small32, n_tok, L.nsmall, W)));
-    const int Rv = a.heads * a.vdim;
-    if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) {
+    const bool diff = L.c.mixer == B200_MIXER_DIFF_ATTENTION;
+    if (diff && L.nsmall && n_tok >= 64) {      // many rows: the same fp32 sums on the tensor cores where the shape allows
+      TIMED(CLS_FOLD, B200_TRY(head_gemm(st, hb, (long long)W, 0, static_cast<const T*>(L.w_small), (long long)W, 0, h->small32, (long long)L.nsmall, 0, n_tok, L.nsmall, W, 1, 1.f,
+                                         h->attn_tc != 0)));
+    } else if (L.nsmall) {
+      TIMED(CLS_FOLD, B200_TRY(small_proj<T>(h, hb, W, L.w_small, nullptr, h->small32, n_tok, L.nsmall, W)));
+    }
+    const int Rv = diff ? L.ob_ld : a.heads * a.vdim;
+    if (diff) {
+      B200_TRY(diff_attention<T>(h, L, n_tok, max_ctx));
+    } else if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) {
       const bool blend = a.v_mix && li != h->vmix_first, keep = a.v_mix && li == h->vmix_first;
       TIMED(CLS_ELEMENTWISE, B200_LAUNCH(attn_rope_cache_kernel<T>, n_tok, 256, (size_t)a.rot_dims * 4 + 4, st, proj, (long long)L.ldp, L.p_q, L.p_k, L.p_v, L.Nq, L.Nk, L.Nv,
                                          a.dim, a.rot_dims / 2, a.rot_pairing == B200_ROT_ADJACENT, L.freq, L.rot_amp, a.scale, h->qkv32, static_cast<T*>(L.kcache),
@@ -1337,17 +1586,19 @@ int step_parallel(b200_dlm* h, int n_tok, int n_want, int max_ctx, float* logits
       TIMED(CLS_ELEMENTWISE, B200_LAUNCH(gated_gelu_kernel<T>, (unsigned)ceil_div64(n, 256), 256, 0, st, proj, (long long)L.ldp, L.p_ffg, L.p_ffu, act, L.c.ff, n));
       TIMED(CLS_LINEAR, B200_TRY(linear<T>(h, act, L.c.ff, L.down, static_cast<T*>(h->ffo), W, n_tok)));
       ffo = static_cast<const T*>(h->ffo);
-    } else if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU) {
+    } else if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU || L.c.mlp == B200_MLP_MOE_SILU_GLU) {
       TIMED(CLS_EXPERTS, B200_TRY(routed_experts_glu<T>(h, L, hb, n_tok)));
       yexp = static_cast<const T*>(h->yexp);
     }
     TIMED(CLS_ELEMENTWISE, B200_LAUNCH(parallel_block_end_kernel<T>, n_tok, 256, 0, st, h->xin, mixo, ffo, yexp, h->moe_w, L.c.top,
-                                       h->trace_layers ? h->trace + (long long)li * stride : nullptr, last ? nullptr : h->layers[li + 1].n1w, hb, W, c.norm_eps));
+                                       h->trace_layers ? h->trace + (long long)li * stride : nullptr, last ? nullptr : h->layers[li + 1].n1w, hb, W, c.norm_eps, c.norm == B200_NORM_LAYER,
+                                       L.c.identity > 0 ? h->moe_idx : (const int*)nullptr, L.c.experts));
   }
   B200_TRY(check_launch("decoder LM layers"));
   if (n_want > 0) {
     T* hf = static_cast<T*>(h->hf);
-    TIMED(CLS_ELEMENTWISE, B200_LAUNCH(rmsnorm_rows_kernel<T>, n_want, 256, 0, st, h->xin, meta + h->off_want, h->fnw, hf, W, c.norm_eps));
+    TIMED(CLS_ELEMENTWISE, if (c.norm == B200_NORM_LAYER) B200_LAUNCH(layernorm_kernel<T>, n_want, 256, 0, st, h->xin, meta + h->off_want, h->fnw, (const float*)nullptr, hf, W, c.norm_eps);
+          else B200_LAUNCH(rmsnorm_rows_kernel<T>, n_want, 256, 0, st, h->xin, meta + h->off_want, h->fnw, hf, W, c.norm_eps));
     if (h->head.tiles) {
       const int ldl = (c.vocab + 7) / 8 * 8;
       TIMED(CLS_LINEAR, B200_TRY(linear<bf16>(h, reinterpret_cast<const bf16*>(hf), W, h->head, h->head_bf, ldl, n_want)));
@@ -1732,6 +1983,16 @@ int b200_dlm_create(const b200_dlm_config* cfg, b200_dlm** out) {
         B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: the rotary ramp wants positive factor, original, fast and slow", i);
       if (l.mixer == B200_MIXER_SIGMOID_ATTENTION) {
         if (a.kv_heads < 1 || a.heads % a.kv_heads) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: attention wants heads a multiple of kv_heads", i);
+      } else if (l.mixer == B200_MIXER_DIFF_ATTENTION) {
+        if (a.kv_heads < 1 || a.heads % a.kv_heads || a.chunk < 0) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: attention wants heads a multiple of kv_heads and no negative chunk", i);
+        if (a.rot_dims > 0 && (a.rot_scaling == B200_ROT_RAMP || (a.rot_scaling == B200_ROT_LINEAR && !(a.rot_factor > 0.f))))
+          B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: the differential attention's rotation is plain, by bands, or linear with a positive factor", i);
+        if (a.kv_from >= 0) {
+          const bool ok = a.kv_from < i && cfg->layers[a.kv_from].mixer == B200_MIXER_DIFF_ATTENTION && cfg->layers[a.kv_from].a.kv_from < 0;
+          const b200_dlm_mixer& s = cfg->layers[ok ? a.kv_from : i].a;
+          if (!ok || s.heads != a.heads || s.kv_heads != a.kv_heads || s.dim != a.dim || s.vdim != a.vdim)
+            B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: kv_from must name an earlier layer with keys and values of its own and equal head counts and sizes", i);
+        }
       } else if (l.mixer == B200_MIXER_RETENTION) {
         if (a.dim > 256 || !a.decay || a.heads > B200_DLM_MAX_DECAY_HEADS) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: retention wants dim in 1..256 and one decay per head", i);
       } else if (l.mixer == B200_MIXER_DELTA) {
@@ -1740,10 +2001,17 @@ int b200_dlm_create(const b200_dlm_config* cfg, b200_dlm** out) {
       } else {
         B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: mixer %d is not registered for this block arrangement", i, l.mixer);
       }
-      if (l.mlp != B200_MLP_NONE && l.mlp != B200_MLP_DENSE_GATED_GELU && l.mlp != B200_MLP_MOE_CLAMPED_GLU)
+      const bool diff = l.mixer == B200_MIXER_DIFF_ATTENTION;
+      if (l.mlp != B200_MLP_NONE && (diff ? l.mlp != B200_MLP_DENSE_CLAMPED_GLU && l.mlp != B200_MLP_MOE_SILU_GLU : l.mlp != B200_MLP_DENSE_GATED_GELU && l.mlp != B200_MLP_MOE_CLAMPED_GLU))
         B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: mlp kind %d is not registered for this block arrangement", i, l.mlp);
       if (l.mlp == B200_MLP_MOE_CLAMPED_GLU && (l.experts < 1 || l.experts > 4096 || l.top < 1 || l.top > l.experts || l.top > 32 || !(l.expert_limit > 0.f)))
         B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: experts in 1..4096, top in 1..min(experts, 32) and a positive limit", i);
+      if (l.mlp == B200_MLP_DENSE_CLAMPED_GLU && !(l.expert_limit > 0.f)) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: the gated unit wants a positive limit", i);
+      if (l.mlp == B200_MLP_MOE_SILU_GLU) {
+        const int n = l.experts + l.identity, groups = l.groups > 1 ? l.groups : 1, keep = groups > 1 ? l.groups_keep : 1;
+        if (l.experts < 1 || l.identity < 0 || l.shared_ff < 0 || n > 4096 || n % groups || keep < 1 || keep > groups || l.top < 1 || l.top > n / groups * keep || l.top > 32)
+          B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: experts + identity in 1..4096, equal groups, and top in 1..32 within the kept groups", i);
+      }
     } else if (cfg->block == B200_BLOCK_GATED_DEPTH_AVERAGE) {
       if (l.mixer != B200_MIXER_LATENT_ATTENTION) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: mixer %d is not registered for this block arrangement", i, l.mixer);
       if (a.heads < 1 || a.dim < 1 || a.vdim < 1 || a.kv_rank < 1 || a.kv_rank > 1024)
@@ -1897,7 +2165,7 @@ int b200_dlm_finalize(b200_dlm* h) {
     L.sig = sig;
   }
   B200_TRY(get_f32(h, "final.norm", W, &h->fnw));
-  if (parallel) B200_LAUNCH(add_one_kernel, ceil_div((int)W, 256), 256, 0, nullptr, h->fnw, (int)W);      // stored around zero
+  if (parallel && c.norm == B200_NORM_RMS_ZERO_CENTRED) B200_LAUNCH(add_one_kernel, ceil_div((int)W, 256), 256, 0, nullptr, h->fnw, (int)W);      // stored around zero
   if (!sandwich && !parallel && !streams) B200_TRY(get_f32(h, "final.norm.b", W, &h->fnb));
   if (c.tied_head) {      // the logits come from the embedding table: its rows stay (the gather), a packed copy serves the product
     h->head.rm = h->embed; h->head.N = c.vocab; h->head.K = (int)W;
@@ -1998,7 +2266,15 @@ int b200_dlm_cache_begin(b200_dlm* h, int slots, int capacity, int max_step_toke
     }
     if (parallel) {
       // per request: keys and values of an attention layer; the matrix memory of a recurrent one and its convolutions' last inputs
-      if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) {
+      if (L.c.mixer == B200_MIXER_DIFF_ATTENTION) {      // a layer that reads another one's keys and values holds none
+        if (a.kv_from < 0) {
+          B200_TRY(A.alloc(&L.kcache, (size_t)slots * capacity * L.Nk * es));
+          B200_TRY(A.alloc(&L.vcache, (size_t)slots * capacity * L.Nv * es));
+        }
+        max_qkv = std::max(max_qkv, (size_t)L.Nq);
+        max_hv = std::max(max_hv, (size_t)L.ob_ld);
+        max_part = std::max(max_part, (size_t)(L.sig_mma >= 0 ? 64 : L.QT) * (2 * a.vdim + 4));
+      } else if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) {
         B200_TRY(A.alloc(&L.kcache, (size_t)slots * capacity * L.Nk * es));
         B200_TRY(A.alloc(&L.vcache, (size_t)slots * capacity * L.Nv * es));
         max_qkv = std::max(max_qkv, (size_t)L.Nq);
@@ -2017,7 +2293,7 @@ int b200_dlm_cache_begin(b200_dlm* h, int slots, int capacity, int max_step_toke
         max_segrow = std::max(max_segrow, (size_t)a.heads * (a.vdim + 1) * a.dim);
         max_heads = std::max(max_heads, (size_t)a.heads);
       }
-      if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU) {
+      if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU || L.c.mlp == B200_MLP_MOE_SILU_GLU) {
         max_e = std::max(max_e, (size_t)L.c.experts); max_top = std::max(max_top, (size_t)L.c.top);
         max_eff = std::max(max_eff, (size_t)L.c.top * L.c.ff);
       }
@@ -2084,6 +2360,7 @@ int b200_dlm_cache_begin(b200_dlm* h, int slots, int capacity, int max_step_toke
       B200_TRY(A.alloc_t(&h->gend, (size_t)h->max_chunks * max_gate));
     }
   } else if (parallel) {
+    for (auto& r : h->rots) B200_TRY(A.alloc_t(&r.table, T * r.m.rot_dims));
     const size_t nseg = (size_t)(max_step_tokens / std::max(h->scan_seg, 8) + 2);
     B200_TRY(A.alloc_t(&h->qkv32, T * max_qkv));
     B200_TRY(A.alloc_t(&h->small32, T * max_small));
@@ -2404,9 +2681,12 @@ int64_t b200_dlm_algorithmic_bytes(b200_dlm* h, int tokens, int context) {
   if (h->cfg.block == B200_BLOCK_PARALLEL_RESIDUAL) {      // `tokens` = requests when decoding, as for the sandwich block
     for (auto& L : h->layers) {
       const b200_dlm_mixer& a = L.c.a;
-      if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) b += ((int64_t)context + tokens) * (L.Nk + L.Nv) * es;      // every cached key and value once
+      if (L.c.mixer == B200_MIXER_DIFF_ATTENTION) {      // every request reads its chunk up to its own position, and writes a row where the layer owns the cache
+        const int64_t per = tokens > 0 ? (int64_t)context / tokens : 0, seen = a.chunk > 0 ? per % a.chunk : per;
+        b += (seen + (a.kv_from < 0 ? 1 : 0)) * tokens * (L.Nk + L.Nv) * es;
+      } else if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) b += ((int64_t)context + tokens) * (L.Nk + L.Nv) * es;      // every cached key and value once
       else b += 2 * (int64_t)tokens * a.heads * a.dim * a.vdim * 4;                                              // the matrix memories, read and written
-      if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU) {
+      if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU || L.c.mlp == B200_MLP_MOE_SILU_GLU) {
         const int64_t used = std::min<int64_t>(L.c.experts, (int64_t)tokens * L.c.top);
         b -= (int64_t)(L.c.experts - used) * 3 * L.c.ff * W * es;
       }
@@ -2452,11 +2732,15 @@ int64_t b200_dlm_algorithmic_flops(b200_dlm* h, int tokens, int context) {
     }
     if (h->cfg.block == B200_BLOCK_PARALLEL_RESIDUAL) {
       const b200_dlm_mixer& a = L.c.a;
-      f += 2 * T * W * L.ncat + 2 * T * W * L.nsmall + 2 * T * W * a.heads * a.vdim;
-      if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) f += 2 * a.heads * (a.dim + a.vdim + a.heads) * (T * context + T * (T + 1) / 2);      // scores, head mix, sums
+      f += 2 * T * W * L.ncat + 2 * T * W * L.nsmall + 2 * T * W * (L.c.mixer == B200_MIXER_DIFF_ATTENTION ? L.ob_ld : a.heads * a.vdim);
+      if (L.c.mixer == B200_MIXER_DIFF_ATTENTION) {
+        int64_t pairs = 0;       // (query, key) pairs of one prompt of T tokens on top of `context`
+        for (int64_t t = 0; t < T; ++t) pairs += (a.chunk > 0 ? (context + t) % a.chunk : context + t) + 1;
+        f += 4 * pairs * a.heads * (a.dim + a.vdim);
+      } else if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) f += 2 * a.heads * (a.dim + a.vdim + a.heads) * (T * context + T * (T + 1) / 2);      // scores, head mix, sums
       else f += (L.c.mixer == B200_MIXER_DELTA ? 8 : 4) * T * a.heads * a.dim * a.vdim;
       if (L.c.mlp == B200_MLP_DENSE_GATED_GELU) f += 2 * T * W * L.c.ff;                   // the down-projection (gate and value are inside ncat)
-      if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU) f += 6 * T * L.c.top * W * L.c.ff;
+      if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU || L.c.mlp == B200_MLP_MOE_SILU_GLU) f += 6 * T * L.c.top * W * L.c.ff;
       continue;
     }
     if (h->cfg.block == B200_BLOCK_SANDWICH) {

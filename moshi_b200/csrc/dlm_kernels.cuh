@@ -32,7 +32,7 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 
 __device__ __forceinline__ float sigmoidf(float z) { return 1.f / (1.f + expf(-z)); }
 
-// layer norm with weight and bias of one fp32 row (two passes: mean, then the mean of squared deviations) -> T
+// layer norm with weight and (when given) bias of one fp32 row (two passes: mean, then the mean of squared deviations) -> T
 template <typename T>
 __device__ __forceinline__ void block_layernorm(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ b,
                                                 T* __restrict__ out, int W, float eps, float* red) {
@@ -42,7 +42,7 @@ __device__ __forceinline__ void block_layernorm(const float* __restrict__ x, con
   float q = 0.f;
   for (int i = threadIdx.x; i < W; i += blockDim.x) { const float d = x[i] - mean; q += d * d; }
   const float rstd = 1.f / sqrtf(block_sum(q, red) / (float)W + eps);
-  for (int i = threadIdx.x; i < W; i += blockDim.x) out[i] = from_f<T>((x[i] - mean) * rstd * w[i] + b[i]);
+  for (int i = threadIdx.x; i < W; i += blockDim.x) out[i] = from_f<T>((x[i] - mean) * rstd * w[i] + (b ? b[i] : 0.f));
 }
 
 // x = table[token] * scale -> the layer-input stream and slot 0 of the per-layer result stack

@@ -1018,7 +1018,8 @@ __global__ void __launch_bounds__(256) sublayer_end_kernel(float* __restrict__ x
 // softmax over those alone.  moe_group_kernel (ONE CTA): sorts the (token, choice) pairs by expert: pos-th row of the grouped
 // order is pair perm[pos] of token row_tok[pos], and cuts every expert's rows into tiles of tile_m for the grouped products
 // (tile -> expert, first row, rows); n_tiles[0] = number of tiles.  The order inside an expert follows the atomics and may
-// differ from run to run; a row's result does not depend on it (every row of a product is summed on its own).
+// differ from run to run; a row's result does not depend on it (every row of a product is summed on its own).  Choices from E
+// on stand for no feed-forward and get no row.
 // ---------------------------------------------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, int E, int top, int* __restrict__ idx,
                                                         float* __restrict__ wts, int n_tok) {
@@ -1056,7 +1057,7 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int* __restrict__
   int* off = cnt + E;
   for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) rank[i] = atomicAdd(&cnt[idx[i]], 1);
+  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) if (idx[i] < E) rank[i] = atomicAdd(&cnt[idx[i]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int o = 0, nt = 0;
@@ -1069,6 +1070,7 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int* __restrict__
   }
   __syncthreads();
   for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
+    if (idx[i] >= E) continue;
     const int pos = off[idx[i]] + rank[i];
     perm[pos] = i;
     row_tok[pos] = i / top;
@@ -1131,7 +1133,7 @@ __global__ void __launch_bounds__(256) grouped_gemm_kernel(const TA* __restrict_
 
 // The same grouped product on the tensor cores (mma.sync m16n8k16, bf16 in, fp32 accumulate): K a multiple of 16, rows of A
 // and B on 16-byte boundaries; act 2: gate and value rows of B alternate and the epilogue writes
-// min(g, limit) * sigmoid(1.702 min(g, limit)) * (clamp(u, -limit, limit) + 1) into column n / 2.  CTA tile 128 x 128 (tiles of 128 rows in the tile table), 8 warps of 32 x 64, 64-element
+// min(g, limit) * sigmoid(1.702 min(g, limit)) * (clamp(u, -limit, limit) + 1) into column n / 2, act 3 silu(g) * u.  CTA tile 128 x 128 (tiles of 128 rows in the tile table), 8 warps of 32 x 64, 64-element
 // k-steps through two shared-memory buffers filled by cp.async (chunks outside M, N or K are zero-filled by a copy of size 0).
 __device__ __forceinline__ void cp_async_16_or_zero(void* smem_dst, const void* src, bool valid) {
   const unsigned d = (unsigned)__cvta_generic_to_shared(smem_dst);
@@ -1212,8 +1214,10 @@ __global__ void __launch_bounds__(256, 2) grouped_gemm_mma_kernel(const bf16* __
       for (int nb = 0; nb < 8; ++nb) {
         const int n = n0 + wn + nb * 8 + 2 * t4;
         float v0 = acc[mf][nb][2 * hf], v1 = acc[mf][nb][2 * hf + 1];
-        if (act == 2) {      // rows of B interleave gate and value: columns (n, n + 1) are one output, column n / 2 of C
-          if (n + 1 < N) {
+        if (act >= 2) {      // rows of B interleave gate and value: columns (n, n + 1) are one output, column n / 2 of C
+          if (n + 1 < N && act == 3) {
+            C[crow * ldc + (n >> 1)] = __float2bfloat16_rn(v0 / (1.f + expf(-v0)) * v1);
+          } else if (n + 1 < N) {
             const float g = fminf(v0, limit), u = fminf(fmaxf(v1, -limit), limit);
             C[crow * ldc + (n >> 1)] = __float2bfloat16_rn(g / (1.f + expf(-1.702f * g)) * (u + 1.f));
           }

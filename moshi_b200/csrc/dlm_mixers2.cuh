@@ -21,11 +21,19 @@ __device__ __forceinline__ float clamped_gluf(float g, float u, float limit) {
   return g * sigmoidf(1.702f * g) * (u + 1.f);
 }
 
-// x = table[token] * scale -> residual stream (fp32);  h = x / sqrt(mean(x^2) + eps) * w1 -> T   (w1 = 1 + the stored weight)
+// the block's norm of one fp32 row -> T: layer norm without a bias, or RMS norm (w = 1 + the stored weight)
+template <typename T>
+__device__ __forceinline__ void block_norm(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ h, int W, float eps, int layer, float* red) {
+  if (layer) { block_layernorm<T>(x, w, nullptr, h, W, eps, red); return; }
+  const float r = block_rrms(x, W, eps, red);
+  for (int i = threadIdx.x; i < W; i += blockDim.x) h[i] = from_f<T>(x[i] * r * w[i]);
+}
+
+// x = table[token] * scale -> residual stream (fp32);  h = norm(x) * w1 -> T
 template <typename T>
 __global__ void __launch_bounds__(256) embed_scale_norm_kernel(const int* __restrict__ tokens, const T* __restrict__ table, int vocab, int W, float scale,
                                                                const float* __restrict__ w1, float* __restrict__ xin, T* __restrict__ h, float eps,
-                                                               int* __restrict__ err) {
+                                                               int* __restrict__ err, int layer) {
   __shared__ float red[32];
   const long long t = blockIdx.x;
   int id = tokens[t];
@@ -35,17 +43,17 @@ __global__ void __launch_bounds__(256) embed_scale_norm_kernel(const int* __rest
   float* x = xin + t * W;
   for (int i = threadIdx.x; i < W; i += blockDim.x) x[i] = bad ? 0.f : to_f(row[i]) * scale;
   __syncthreads();
-  const float r = block_rrms(x, W, eps, red);
-  for (int i = threadIdx.x; i < W; i += blockDim.x) h[t * W + i] = from_f<T>(x[i] * r * w1[i]);
+  block_norm<T>(x, w1, h + t * W, W, eps, layer, red);
 }
 
 // End of a parallel block, one CTA per token:  x <- x + mix + ff,  ff = a dense feed-forward's row | sum_k ew[t][k] * rows of
-// the chosen experts | nothing;  optional copy of x (per-layer trace);  optional h = rms_norm(x) * w_next for the next layer.
+// the chosen experts (the row of h itself for a choice from n_exp on: an identity expert) | both | nothing;  optional copy of x
+// (per-layer trace);  optional h = norm(x) * w_next for the next layer.
 template <typename T>
 __global__ void __launch_bounds__(256) parallel_block_end_kernel(float* __restrict__ xin, const T* __restrict__ mix, const T* __restrict__ ff,
                                                                  const T* __restrict__ yexp, const float* __restrict__ ew, int top,
-                                                                 float* __restrict__ trace, const float* __restrict__ w_next, T* __restrict__ h,
-                                                                 int W, float eps) {
+                                                                 float* __restrict__ trace, const float* __restrict__ w_next, T* h,
+                                                                 int W, float eps, int layer = 0, const int* __restrict__ choice = nullptr, int n_exp = 0) {
   __shared__ float red[32];
   const long long t = blockIdx.x;
   float* x = xin + t * W;
@@ -54,7 +62,10 @@ __global__ void __launch_bounds__(256) parallel_block_end_kernel(float* __restri
     if (ff) y += to_f(ff[t * W + i]);
     if (yexp) {
       float acc = 0.f;
-      for (int k = 0; k < top; ++k) acc = fmaf(ew[t * top + k], to_f(yexp[(t * top + k) * W + i]), acc);
+      for (int k = 0; k < top; ++k) {
+        const bool self = choice && choice[t * top + k] >= n_exp;
+        acc = fmaf(ew[t * top + k], to_f(self ? h[t * W + i] : yexp[(t * top + k) * W + i]), acc);
+      }
       y += acc;
     }
     const float v = x[i] + y;
@@ -63,8 +74,7 @@ __global__ void __launch_bounds__(256) parallel_block_end_kernel(float* __restri
   }
   if (w_next) {
     __syncthreads();
-    const float r = block_rrms(x, W, eps, red);
-    for (int i = threadIdx.x; i < W; i += blockDim.x) h[t * W + i] = from_f<T>(x[i] * r * w_next[i]);
+    block_norm<T>(x, w_next, h + t * W, W, eps, layer, red);
   }
 }
 
@@ -806,13 +816,15 @@ __global__ void __launch_bounds__(256) gated_gelu_kernel(const T* __restrict__ p
   out[i] = from_f<T>(gelu_tanhf(to_f(proj[t * ldp + off_gate + f])) * to_f(proj[t * ldp + off_up + f]));
 }
 
-// out[r][f] = clamped_glu(in[r][2f], in[r][2f + 1]): the experts' first product with gate and value rows interleaved
+// out[r][f] = clamped_glu(in[r][2f], in[r][2f + 1]), or silu(in[r][2f]) * in[r][2f + 1]: the experts' first product with gate and
+// value rows interleaved
 template <typename T>
-__global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ in, T* __restrict__ out, int F, long long n, float limit) {
+__global__ void __launch_bounds__(256) interleaved_glu_kernel(const T* __restrict__ in, T* __restrict__ out, int F, long long n, float limit, int silu) {
   const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
   if (i >= n) return;
   const long long r = i / F; const int f = (int)(i - r * F);
-  out[i] = from_f<T>(clamped_gluf(to_f(in[r * 2 * F + 2 * f]), to_f(in[r * 2 * F + 2 * f + 1]), limit));
+  const float g = to_f(in[r * 2 * F + 2 * f]), u = to_f(in[r * 2 * F + 2 * f + 1]);
+  out[i] = from_f<T>(silu ? g * sigmoidf(g) * u : clamped_gluf(g, u, limit));
 }
 
 // Router with sigmoid scores, per token (one warp): s = sigmoid(logit); the `top` experts with the largest s + correction are

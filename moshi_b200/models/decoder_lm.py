@@ -12,7 +12,7 @@ import typing as tp
 import torch
 
 from .. import _lib
-from ..config import BLOCKS, MIXERS, MLP_KINDS, ROT_PAIRINGS, ROT_SCALINGS, SINKS, DecoderLMConfig, MixerConfig
+from ..config import BLOCKS, MIXERS, MLP_KINDS, NORMS, ROT_PAIRINGS, ROT_SCALINGS, SINKS, DecoderLMConfig, MixerConfig
 
 _DTYPES = {torch.bfloat16: _lib.B200_BF16, torch.float32: _lib.B200_F32}
 
@@ -28,6 +28,7 @@ def _fill_mixer(dst, m: MixerConfig) -> None:
     dst.rot_fast, dst.rot_slow = float(sc.get("fast", 0.0)), float(sc.get("slow", 0.0))
     dst.softcap, dst.v_mix = m.softcap, int(m.v_mix)
     dst.bias, dst.sink, dst.head_gate = int(m.bias), SINKS[m.sink], int(m.head_gate)
+    dst.chunk, dst.qk_norm, dst.diff, dst.kv_from = m.chunk, int(m.qk_norm), m.diff, m.kv_from
     if m.decay:
         dst.decay = (C.c_float * len(m.decay))(*m.decay)      # ctypes keeps the array alive with the struct; create() copies it
 
@@ -55,6 +56,7 @@ class DecoderLM:
             layers[i].experts, layers[i].top = L.experts, L.top
             layers[i].expert_limit, layers[i].router_scale = L.expert_limit, L.router_scale
             layers[i].a_scale, layers[i].b_scale = L.a_scale, L.b_scale
+            layers[i].shared_ff, layers[i].identity, layers[i].groups, layers[i].groups_keep = L.shared_ff, L.identity, L.groups, L.groups_keep
             for dst, m in zip((layers[i].a, layers[i].b), L.mixers()):
                 if m is not None:
                     _fill_mixer(dst, m)
@@ -63,6 +65,7 @@ class DecoderLM:
         c.embedding_scale, c.residual_mult, c.norm_eps = cfg.embedding_scale, cfg.residual_mult, cfg.norm_eps
         c.block, c.canon_taps, c.logit_softcap = BLOCKS[cfg.block], cfg.canon_taps, cfg.logit_softcap
         c.streams, c.logit_scale, c.tied_head = cfg.streams, cfg.logit_scale, int(cfg.tied_head)
+        c.norm = NORMS[cfg.norm]
         c.compute_dtype = _DTYPES[dtype]
         c.layers = layers
         items = tensors.items() if isinstance(tensors, tp.Mapping) else tensors

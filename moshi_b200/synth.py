@@ -275,7 +275,7 @@ def iter_synth_decoder_tensors(cfg: DecoderLMConfig, seed: int = 99, device="cpu
     sit around 1, biases and sinks around 0, and the depth-average rows are positive and sum to 1, so that activations keep a
     sane scale through any number of layers."""
     gen = _gen(seed, device)
-    zero_centred = cfg.block == "parallel_residual"          # norm weights stored around zero (the norm multiplies by 1 + w)
+    zero_centred = cfg.block == "parallel_residual" and cfg.norm == "rms_zero_centred"          # norm weights stored around zero (the norm multiplies by 1 + w)
     for name, shape in cfg.tensor_shapes().items():
         leaf = name.split(".", 1)[-1] if name.startswith("l") and name[1].isdigit() else name
         last = leaf.rsplit(".", 1)[-1]
