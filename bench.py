@@ -1053,6 +1053,121 @@ def dibulix_arm(args) -> None:
     print(json.dumps(out))
 
 
+# ---------------------------------------------------------------------------------------------
+# --decoder-lm --decoder-arch megolorn: the Megolorn design beside a Namalix model (the closest existing one: parallel blocks with
+# attention, dense and routed gated feed-forwards on the same handle and step) of equal width, depth, head counts, projection
+# sizes, feed-forwards, experts and vocabulary
+# ---------------------------------------------------------------------------------------------
+MEGOLORN_SIZES = {
+    # name: (width, layers, heads, kv heads, map dim, value dim, chunk, experts, top, expert ff, shared ff, dense ff, vocab)
+    "w2048": (2048, 4, 16, 4, 64, 128, 8192, 16, 2, 4096, 4096, 8192, 32000),
+    "w4096": (4096, 2, 32, 8, 64, 128, 8192, 16, 2, 8192, 8192, 16384, 32000),
+}
+
+
+def _megolorn_cfgs(size: str) -> dict:
+    from moshi_b200.config import DecoderLMConfig
+    W, n, H, G, d, dv, chunk, E, top, ff, sff, dff, V = MEGOLORN_SIZES[size]
+
+    def meg(chunk):
+        mixer = {"diff": 0.5, "dim": d, "heads": H, "kv_heads": G, "mask": {"size": chunk}, "rot": {"base": 5e5, "dims": d, "scaling": {"factor": 8.0}},
+                 "scale": d ** -0.5, "vdim": dv}
+        moe = {"expert": {"ff": ff}, "kind": "moe", "router": {"experts": E, "groups": {"count": 4, "keep": 2}, "identity": 0, "top": top}, "shared": {"ff": sff}}
+        return DecoderLMConfig.from_dict({"architecture": "Megolorn", "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "vocab": V, "width": W, "layers": [
+            {"type": "attention", "mixer": dict(mixer, kv_from=i - 1) if i % 2 else mixer, "mlp": moe if i % 2 else {"ff": dff, "kind": "dense", "limit": 7.0}}
+            for i in range(n)]})
+    nam = {"dim": 2 * d, "heads": H, "kv_heads": G, "scale": (2 * d) ** -0.5, "softcap": 50.0, "v_mix": False, "vdim": dv, "rot": {"base": 5e5, "dims": d}}
+    nmoe = {"expert": {"ff": ff, "limit": 7.0}, "kind": "moe", "router": {"experts": E, "scale": 2.0, "top": top}}
+    return {"megolorn": meg(chunk), "megolorn_chunk_1024": meg(1024),
+            "namalix_equal": DecoderLMConfig.from_dict({"architecture": "Namalix", "embedding": {"scale": W ** 0.5}, "norm": {"eps": 1e-6}, "vocab": V, "width": W, "layers": [
+                {"type": "attention", "mixer": nam, "mlp": nmoe if i % 2 else {"ff": dff, "kind": "dense"}} for i in range(n)]})}
+
+
+def megolorn_arm(args) -> None:
+    """Prefill (one prompt of --prefill-tokens) and decode (--decode-batch requests, one token each, on --context cached tokens)
+    of the Megolorn design with random weights, per size: whole steps and per class of kernel, beside the like classes of a Namalix
+    model of equal sizes, against the measured rooflines."""
+    from moshi_b200 import _lib
+    from moshi_b200.models import DecoderLMGen, loaders
+    device = torch.device("cuda:0")
+    torch.cuda.set_device(device)
+    hbm, src = _peaks()
+    pk = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
+    tf = float(pk.get("bf16_tflops", 1590.0))
+    T, B, ctx = args.prefill_tokens, args.decode_batch, args.context
+    g = torch.Generator().manual_seed(7)
+    out = {"impl": "b200", "mode": "decoder-lm", "arch": "megolorn", "dtype": "bf16", "data": "synthetic (random weights)",
+           "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src}, "workload": {"prefill_tokens": T, "decode_batch": B, "context": ctx}, "sizes": {}}
+    launches0 = _lib.lib().b200_launch_count()
+
+    def measure(cfg):
+        model = loaders.get_decoder_lm(None, cfg, device=device, synth_seed=11)
+        gen = DecoderLMGen(model, slots=B, capacity=ctx + 64, max_step_tokens=max(T, B), max_want=B)
+        V = cfg.vocab
+        prompt = torch.randint(0, V, (T,), generator=g).tolist()
+
+        def prefill():
+            gen.step([(0, prompt)], [T - 1])
+            gen.release(0)
+
+        def classes(fn):
+            gen.set_option("time_kernels", 1)
+            gen.kernel_times()
+            for _ in range(3):
+                fn()
+            kt = {k: v / 3 for k, v in gen.kernel_times().items()}
+            gen.set_option("time_kernels", 0)
+            return kt
+        W, n, H, G, d, dv, _, E, top, ff, sff, dff, _ = MEGOLORN_SIZES[size]
+        meg = cfg.architecture == "Megolorn"
+        n_moe, n_dense, chunk = n // 2, (n + 1) // 2, cfg.layers[0].a.chunk
+        # matrix products of the layers: q | k | v (keys and values in every other layer here), gated units, output products
+        wq, wkv, wo = 2 * H * d * W, G * (2 * d + dv) * W, H * dv * W
+        lin = n * (wq + wo) + (n_dense if meg else n) * wkv + n_dense * 3 * dff * W + (n_moe * 3 * sff * W if meg else 0)
+        pairs = sum((t % chunk if chunk else t) + 1 for t in range(T))
+        attn_fl = n * 2 * pairs * H * (2 * d + (2 if meg else 1) * dv)      # both maps' scores; the sums of both maps
+        exp_fl = n_moe * 6 * T * top * W * ff
+        res = {"prefill": {"ms": _timed_steps(prefill, args.steps, args.warmup)}}
+        kt = classes(prefill)
+        res["prefill"].update({"tokens_per_s": T / res["prefill"]["ms"] * 1e3, "kernel_ms": kt, "tflops": (2 * T * lin + attn_fl + exp_fl) / res["prefill"]["ms"] / 1e9,
+                               "kernel_frac_of_bf16_peak": {"linear": 2 * T * lin / kt["linear"] / 1e9 / tf, "attention": attn_fl / kt["attention"] / 1e9 / tf,
+                                                            "experts": exp_fl / kt["experts"] / 1e9 / tf}})
+        filler = torch.randint(0, V, (ctx,), generator=g).tolist()
+        for b in range(B):
+            for a in range(0, ctx, max(T, B)):
+                gen.step([(b, filler[a:a + max(T, B)])], [])
+        toks = torch.randint(0, V, (B,), generator=g).tolist()
+        # every request's position goes up by one per step, as in serving; a chunked layer starts a new chunk where one ends
+        start = gen.slot_length(0)
+
+        def decode():
+            gen.step([(b, [toks[b]]) for b in range(B)], list(range(B)))
+        res["decode"] = {"ms": _timed_steps(decode, min(args.steps, 40), min(args.warmup, 5))}
+        kt = classes(decode)
+        seen = (start % chunk if chunk else start) + min(args.steps, 40)
+        attn_bytes = n * B * seen * G * (2 * d + dv) * 2
+        exp_bytes = n_moe * min(E, B * top) * 3 * ff * W * 2
+        lin_bytes = (lin + V * W) * 2
+        nbytes = attn_bytes + exp_bytes + lin_bytes
+        res["decode"].update({"tokens_per_s": B / res["decode"]["ms"] * 1e3, "kernel_ms": kt, "algorithmic_bytes": nbytes, "frac_of_hbm_peak": nbytes / res["decode"]["ms"] / 1e6 / hbm,
+                              "kernel_frac_of_hbm_peak": {"linear": lin_bytes / kt["linear"] / 1e6 / hbm, "attention": attn_bytes / kt["attention"] / 1e6 / hbm,
+                                                          "experts": exp_bytes / kt["experts"] / 1e6 / hbm}})
+        assert gen.error_flags() == 0
+        gen.close()
+        del gen, model
+        torch.cuda.empty_cache()
+        return res
+
+    for size in args.decoder_sizes.split(","):
+        res = {"config": dict(zip(("width", "layers", "heads", "kv_heads", "map_dim", "value_dim", "chunk", "experts", "top", "expert_ff", "shared_ff", "dense_ff", "vocab"),
+                                  MEGOLORN_SIZES[size])), "models": {}}
+        for name, cfg in _megolorn_cfgs(size).items():
+            res["models"][name] = measure(cfg)
+        out["sizes"][size] = res
+    out["gpu_launches"] = int(_lib.lib().b200_launch_count() - launches0)
+    print(json.dumps(out))
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1070,17 +1185,18 @@ def main() -> None:
     ap.add_argument("--decoder-lm", action="store_true",
                     help="instead of the default workload: prefill / decode throughput of the text-only decoder LM (Likosun design, random "
                          "weights) beside the Moshi temporal transformer at equal width and depth; prints its own JSON line")
-    ap.add_argument("--decoder-arch", choices=["likosun", "govuvik", "namalix", "dibulix"], default="likosun",
+    ap.add_argument("--decoder-arch", choices=["likosun", "govuvik", "namalix", "dibulix", "megolorn"], default="likosun",
                     help="with --decoder-lm: which design to time (govuvik: window attention beside gated linear attention, mLSTM, routed experts; "
                          "namalix: sigmoid attention, retention, delta rule, clamped routed experts; dibulix: residual streams, latent attention "
-                         "with a rotated key part, window attention beside a minGRU, delta rule with a decay per key channel)")
+                         "with a rotated key part, window attention beside a minGRU, delta rule with a decay per key channel; megolorn: differential attention "
+                         "on chunks, softmax-routed experts with groups and a shared expert)")
     ap.add_argument("--decoder-sizes", default="w2048,w4096", help="comma-separated names out of " + ",".join(DECODER_SIZES))
     ap.add_argument("--prefill-tokens", type=int, default=2048)
     ap.add_argument("--decode-batch", type=int, default=32)
     ap.add_argument("--context", type=int, default=2048)
     args = ap.parse_args()
     if args.decoder_lm:
-        {"govuvik": govuvik_arm, "namalix": namalix_arm, "dibulix": dibulix_arm}.get(args.decoder_arch, decoder_lm_arm)(args)
+        {"govuvik": govuvik_arm, "namalix": namalix_arm, "dibulix": dibulix_arm, "megolorn": megolorn_arm}.get(args.decoder_arch, decoder_lm_arm)(args)
         return
     if args.impl == "reference":
         reference_arm(args)
