@@ -1061,7 +1061,7 @@ def dibulix_arm(args) -> None:
 MEGOLORN_SIZES = {
     # name: (width, layers, heads, kv heads, map dim, value dim, chunk, experts, top, expert ff, shared ff, dense ff, vocab)
     "w2048": (2048, 4, 16, 4, 64, 128, 8192, 16, 2, 4096, 4096, 8192, 32000),
-    "w4096": (4096, 2, 32, 8, 64, 128, 8192, 16, 2, 8192, 8192, 16384, 32000),
+    "w4096": (4096, 2, 16, 4, 64, 128, 8192, 16, 2, 8192, 8192, 16384, 32000),
 }
 
 

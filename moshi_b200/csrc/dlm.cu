@@ -624,7 +624,16 @@ int finalize_sandwich_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
 
 template <typename T>
 int small_proj(b200_dlm* h, const T* x, long long ldx, const void* w, const float* b, float* out, int M, int N, int K) {
-  B200_LAUNCH(small_proj_f32_kernel<T>, M, 256, (size_t)K * 4, h->stream, x, ldx, static_cast<const T*>(w), b, out, N, K);
+  static bool attr_set = false;
+  if (!attr_set) {
+    B200_CUDA(cudaFuncSetAttribute((small_proj_f32_kernel<T, 1>), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    B200_CUDA(cudaFuncSetAttribute((small_proj_f32_kernel<T, 8>), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    attr_set = true;
+  }
+  const int vec = K % 8 == 0 && (ldx * sizeof(T)) % 16 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0;
+  const size_t row = (size_t)K * sizeof(T);
+  if (M >= 512 && 8 * row <= 100 * 1024) B200_LAUNCH((small_proj_f32_kernel<T, 8>), dim3(ceil_div(M, 8), ceil_div(N, 32)), 256, 8 * row, h->stream, x, ldx, static_cast<const T*>(w), b, out, M, N, K, vec);
+  else B200_LAUNCH((small_proj_f32_kernel<T, 1>), dim3(M, M >= 512 ? 1 : ceil_div(N, 8)), 256, row, h->stream, x, ldx, static_cast<const T*>(w), b, out, M, N, K, vec);
   return check_launch("small_proj_f32");
 }
 
@@ -1356,7 +1365,8 @@ int diff_attention(b200_dlm* h, const Layer& L, int n_tok, int max_ctx) {
     p.kcache = S.kcache; p.vcache = S.vcache; p.cap = h->cap; p.tok_slot = h->meta_dev + h->off_slot; p.tok_pos = h->meta_dev + h->off_pos;
     p.off_g = L.p_ffg; p.off_u = L.p_ffu; p.F = L.glu_ff; p.glu = L.c.mlp == B200_MLP_DENSE_CLAMPED_GLU ? GLU_CLAMPED : GLU_SILU; p.limit = L.c.expert_limit;
     p.act = static_cast<T*>(h->obuf) + L.ob_act; p.lda = L.ob_ld;
-    const dim3 grid(n_tok, 1 + ceil_div(L.glu_ff, GLU_SLICE));
+    p.head_rows = n_tok >= 512 ? 1 : ceil_div(p.Hm + (own ? p.Gm : 0), 8);      // few tokens: one (head, map) per warp
+    const dim3 grid(n_tok, p.head_rows + ceil_div(L.glu_ff, GLU_SLICE));
     const size_t smem = (size_t)8 * a.dim * sizeof(float);
     TIMED(CLS_ELEMENTWISE, if (mma) B200_LAUNCH((diff_prep_kernel<T, bf16>), grid, 256, smem, st, p); else B200_LAUNCH((diff_prep_kernel<T, float>), grid, 256, smem, st, p));
     B200_TRY(check_launch("diff_prep"));
@@ -1534,12 +1544,7 @@ int step_parallel(b200_dlm* h, int n_tok, int n_want, int max_ctx, float* logits
     const bool last = li + 1 == c.n_layers;
     TIMED(CLS_LINEAR, B200_TRY(linear<T>(h, hb, W, L.cat, proj, L.ldp, n_tok)));
     const bool diff = L.c.mixer == B200_MIXER_DIFF_ATTENTION;
-    if (diff && L.nsmall && n_tok >= 64) {      // many rows: the same fp32 sums on the tensor cores where the shape allows
-      TIMED(CLS_FOLD, B200_TRY(head_gemm(st, hb, (long long)W, 0, static_cast<const T*>(L.w_small), (long long)W, 0, h->small32, (long long)L.nsmall, 0, n_tok, L.nsmall, W, 1, 1.f,
-                                         h->attn_tc != 0)));
-    } else if (L.nsmall) {
-      TIMED(CLS_FOLD, B200_TRY(small_proj<T>(h, hb, W, L.w_small, nullptr, h->small32, n_tok, L.nsmall, W)));
-    }
+    if (L.nsmall) TIMED(CLS_FOLD, B200_TRY(small_proj<T>(h, hb, W, L.w_small, nullptr, h->small32, n_tok, L.nsmall, W)));
     const int Rv = diff ? L.ob_ld : a.heads * a.vdim;
     if (diff) {
       B200_TRY(diff_attention<T>(h, L, n_tok, max_ctx));
@@ -1590,7 +1595,8 @@ int step_parallel(b200_dlm* h, int n_tok, int n_want, int max_ctx, float* logits
       TIMED(CLS_EXPERTS, B200_TRY(routed_experts_glu<T>(h, L, hb, n_tok)));
       yexp = static_cast<const T*>(h->yexp);
     }
-    TIMED(CLS_ELEMENTWISE, B200_LAUNCH(parallel_block_end_kernel<T>, n_tok, 256, 0, st, h->xin, mixo, ffo, yexp, h->moe_w, L.c.top,
+    auto block_end = n_tok <= 592 && W <= 4096 ? parallel_block_end_kernel<T, true> : parallel_block_end_kernel<T, false>;
+    TIMED(CLS_ELEMENTWISE, B200_LAUNCH(block_end, n_tok, 256, 0, st, h->xin, mixo, ffo, yexp, h->moe_w, L.c.top,
                                        h->trace_layers ? h->trace + (long long)li * stride : nullptr, last ? nullptr : h->layers[li + 1].n1w, hb, W, c.norm_eps, c.norm == B200_NORM_LAYER,
                                        L.c.identity > 0 ? h->moe_idx : (const int*)nullptr, L.c.experts));
   }

@@ -521,23 +521,74 @@ __global__ void rows_from_f32_kernel(const float* __restrict__ in, T* __restrict
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
-// Small projections whose result must be fp32 (gates of a recurrence, router logits): out[t][n] = x[t] . w[n] + b[n], one CTA
-// per token, the row in shared memory, one warp per output.  The sum over k has a fixed order whatever else is in the step.
+// Small projections whose result must be fp32 (gates of a recurrence, router logits): out[t][n] = x[t] . w[n] + b[n].  A CTA takes
+// TOK tokens (their rows in shared memory) and, over grid.y, every gridDim.y-th group of eight outputs, one warp per output: many
+// tokens share a read of the weights, few tokens spread over the GPU.  The sum over k has the same order in every layout: a lane
+// adds runs of eight elements (single elements where rows do not start on 16 bytes), then the lanes meet.
 // ---------------------------------------------------------------------------------------------------------------------------
-template <typename T>
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) {
+  const uint4 a = *reinterpret_cast<const uint4*>(p);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&a);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h[i]); v[2 * i] = f.x; v[2 * i + 1] = f.y; }
+}
+
+template <typename T, int TOK>
 __global__ void __launch_bounds__(256) small_proj_f32_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, const float* __restrict__ b,
-                                                             float* __restrict__ out, int N, int K) {
-  extern __shared__ float xrow[];
-  const long long t = blockIdx.x;
-  for (int i = threadIdx.x; i < K; i += blockDim.x) xrow[i] = to_f(x[t * ldx + i]);
+                                                             float* __restrict__ out, int M, int N, int K, int vec) {
+  extern __shared__ __align__(16) unsigned char sp_smem[];
+  T* xs = reinterpret_cast<T*>(sp_smem);                 // [TOK][K]
+  const long long t0 = (long long)blockIdx.x * TOK;
+  const int nt = (int)min((long long)TOK, M - t0);
+  if (vec) {
+    constexpr int E = 16 / (int)sizeof(T);
+    const int kv = K / E;
+    for (int i = threadIdx.x; i < nt * kv; i += 256) {
+      const int r = i / kv, e = i - r * kv;
+      reinterpret_cast<uint4*>(xs)[i] = *reinterpret_cast<const uint4*>(x + (t0 + r) * ldx + (long long)e * E);
+    }
+  } else {
+    for (int i = threadIdx.x; i < nt * K; i += 256) { const int r = i / K; xs[i] = x[(t0 + r) * ldx + (i - r * K)]; }
+  }
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int n = warp; n < N; n += 8) {
+  for (int n = blockIdx.y * 8 + warp; n < N; n += gridDim.y * 8) {
     const T* wr = w + (long long)n * K;
-    float acc = 0.f;
-    for (int k = lane; k < K; k += 32) acc = fmaf(xrow[k], to_f(wr[k]), acc);
-    acc = warp_sum(acc);
-    if (lane == 0) out[t * N + n] = acc + (b ? b[n] : 0.f);
+    float acc[TOK];
+#pragma unroll
+    for (int r = 0; r < TOK; ++r) acc[r] = 0.f;
+    if (vec) {
+#pragma unroll 4
+      for (int k = lane * 8; k < K; k += 256) {
+        float wv[8];
+        load8(wr + k, wv);
+#pragma unroll
+        for (int r = 0; r < TOK; ++r) {
+          if (r < nt) {
+            float xv[8];
+            load8(xs + r * K + k, xv);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) acc[r] = fmaf(xv[e], wv[e], acc[r]);
+          }
+        }
+      }
+    } else {
+      for (int k = lane; k < K; k += 32) {
+        const float wv = to_f(wr[k]);
+#pragma unroll
+        for (int r = 0; r < TOK; ++r)
+          if (r < nt) acc[r] = fmaf(to_f(xs[r * K + k]), wv, acc[r]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < TOK; ++r) {
+      const float s = warp_sum(acc[r]);
+      if (lane == 0 && r < nt) out[(t0 + r) * N + n] = s + (b ? b[n] : 0.f);
+    }
   }
 }
 

@@ -49,7 +49,9 @@ __global__ void __launch_bounds__(256) embed_scale_norm_kernel(const int* __rest
 // End of a parallel block, one CTA per token:  x <- x + mix + ff,  ff = a dense feed-forward's row | sum_k ew[t][k] * rows of
 // the chosen experts (the row of h itself for a choice from n_exp on: an identity expert) | both | nothing;  optional copy of x
 // (per-layer trace);  optional h = norm(x) * w_next for the next layer.
-template <typename T>
+// REG (few tokens, W <= 4096): the row stays in registers between the sum and the norm, which shortens the chain of a CTA; many tokens
+// fill the SMs better with the smaller kernel.
+template <typename T, bool REG>
 __global__ void __launch_bounds__(256) parallel_block_end_kernel(float* __restrict__ xin, const T* __restrict__ mix, const T* __restrict__ ff,
                                                                  const T* __restrict__ yexp, const float* __restrict__ ew, int top,
                                                                  float* __restrict__ trace, const float* __restrict__ w_next, T* h,
@@ -57,7 +59,7 @@ __global__ void __launch_bounds__(256) parallel_block_end_kernel(float* __restri
   __shared__ float red[32];
   const long long t = blockIdx.x;
   float* x = xin + t * W;
-  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+  auto updated = [&](int i) {
     float y = to_f(mix[t * W + i]);
     if (ff) y += to_f(ff[t * W + i]);
     if (yexp) {
@@ -68,7 +70,40 @@ __global__ void __launch_bounds__(256) parallel_block_end_kernel(float* __restri
       }
       y += acc;
     }
-    const float v = x[i] + y;
+    return x[i] + y;
+  };
+  if constexpr (REG) {
+    constexpr int NR = 16;
+    float v[NR], s = 0.f;
+#pragma unroll
+    for (int k = 0; k < NR; ++k) {
+      const int i = threadIdx.x + 256 * k;
+      v[k] = i < W ? updated(i) : 0.f;
+    }
+#pragma unroll
+    for (int k = 0; k < NR; ++k) {
+      const int i = threadIdx.x + 256 * k;
+      if (i >= W) break;
+      x[i] = v[k];
+      if (trace) trace[t * W + i] = v[k];
+      s += v[k];
+    }
+    if (!w_next) return;
+    const float mean = layer ? block_sum(s, red) / (float)W : 0.f;
+    float q = 0.f;
+#pragma unroll
+    for (int k = 0; k < NR; ++k)
+      if (threadIdx.x + 256 * k < W) { const float d = v[k] - mean; q = fmaf(d, d, q); }
+    const float r = 1.f / sqrtf(block_sum(q, red) / (float)W + eps);
+#pragma unroll
+    for (int k = 0; k < NR; ++k) {
+      const int i = threadIdx.x + 256 * k;
+      if (i < W) h[t * W + i] = from_f<T>((v[k] - mean) * r * w_next[i]);
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    const float v = updated(i);
     x[i] = v;
     if (trace) trace[t * W + i] = v;
   }

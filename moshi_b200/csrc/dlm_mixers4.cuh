@@ -27,9 +27,9 @@ __device__ __forceinline__ float gated_unit(float g, float u, int kind, float li
 
 // ---------------------------------------------------------------------------------------------------------------------------
 // Preparation of the attention and of the gated feed-forward beside it, on the concatenated projection proj T [tokens][ld].
-// grid (tokens, 1 + slices).  Row 0 of the grid, one warp per (head, map): x + bias, / rms over dim * w (when w is given), rotated,
+// grid (tokens, head_rows + slices).  The first head_rows rows of the grid, one warp per (head, map): x + bias, / rms over dim * w (when w is given), rotated,
 // queries times qscale -> qout TQ [tokens][Hm * dim], keys -> cache row (off_k < 0: the layer has no keys and values); values +
-// bias -> cache row.  Rows from 1 on: act[:, col] = gated_unit(proj[off_g + col], proj[off_u + col]) on GLU_SLICE columns each.
+// bias -> cache row.  The rows after them: act[:, col] = gated_unit(proj[off_g + col], proj[off_u + col]) on GLU_SLICE columns each.
 // ---------------------------------------------------------------------------------------------------------------------------
 constexpr int GLU_SLICE = 2048;
 
@@ -46,6 +46,7 @@ struct DiffPrepParams {
   const int *tok_slot, *tok_pos;
   int off_g, off_u, F, glu; float limit;
   void* act; long long lda;             // T
+  int head_rows;
 };
 
 template <typename T, typename TQ>
@@ -53,8 +54,8 @@ __global__ void __launch_bounds__(256) diff_prep_kernel(DiffPrepParams p) {
   extern __shared__ float prep_buf[];   // [8 warps][dim]
   const long long t = blockIdx.x;
   const T* row = static_cast<const T*>(p.proj) + t * p.ld;
-  if (blockIdx.y > 0) {
-    const int c0 = ((int)blockIdx.y - 1) * GLU_SLICE, c1 = min(p.F, c0 + GLU_SLICE);
+  if ((int)blockIdx.y >= p.head_rows) {
+    const int c0 = ((int)blockIdx.y - p.head_rows) * GLU_SLICE, c1 = min(p.F, c0 + GLU_SLICE);
     T* act = static_cast<T*>(p.act) + t * p.lda;
     if (sizeof(T) == 2 && ((p.F | p.off_g | p.off_u) & 7) == 0 && ((p.ld | p.lda) & 7) == 0 && ((uintptr_t)p.act & 15) == 0) {
       for (int c = c0 + threadIdx.x * 8; c < c1; c += 256 * 8) {
@@ -80,7 +81,7 @@ __global__ void __launch_bounds__(256) diff_prep_kernel(DiffPrepParams p) {
   const long long crow = (long long)p.tok_slot[t] * p.cap + p.tok_pos[t];
   float* buf = prep_buf + warp * dim;
   const int n = p.Hm + (p.off_k >= 0 ? p.Gm : 0);
-  for (int hm = warp; hm < n; hm += 8) {
+  for (int hm = blockIdx.y * 8 + warp; hm < n; hm += p.head_rows * 8) {
     const bool key = hm >= p.Hm;
     const int i = key ? hm - p.Hm : hm;
     const T* src = row + (key ? p.off_k : p.off_q) + i * dim;
@@ -106,7 +107,7 @@ __global__ void __launch_bounds__(256) diff_prep_kernel(DiffPrepParams p) {
     }
     __syncwarp();
   }
-  if (p.off_k >= 0) {
+  if (p.off_k >= 0 && blockIdx.y == 0) {
     T* vc = static_cast<T*>(p.vcache) + crow * p.Nv;
     const float* b = p.bias ? p.bias + (p.Hm + p.Gm) * dim : nullptr;
     for (int e = threadIdx.x; e < p.Nv; e += 256) vc[e] = from_f<T>(to_f(row[p.off_v + e]) + (b ? b[e] : 0.f));
@@ -296,6 +297,11 @@ __global__ void __launch_bounds__(128) diff_attn_merge_kernel(DiffAttnParams p) 
 // running maxima of their own that meet in shared memory at the end.
 // ---------------------------------------------------------------------------------------------------------------------------
 constexpr int DA_KT = 64;
+__device__ __forceinline__ float exp2_approx(float x) {      // the hardware exponential (2 ulp; results below the normal range become 0)
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 inline size_t diff_attn_mma_smem(int dim, int VT, bool sk) {
   const size_t qs = 2 * dim + 8, vs = VT * 16 + 8, mr = sk ? 16 : 64;
   const size_t tiles = 2 * (mr * qs + 2 * DA_KT * qs + 2 * DA_KT * vs);
@@ -323,19 +329,25 @@ __global__ void __launch_bounds__(128, 2) diff_attn_mma_kernel(DiffAttnParams p)
   const int n_kt = (kmax - kmin) / KT + 1, per = (n_kt + p.nsplit - 1) / p.nsplit;
   const int kt0 = split * per, kt1 = min(n_kt, kt0 + per);
 
+  const int kw = D2 / 8, kdj = 128 / kw, kde = 128 - kdj * kw, kj0 = threadIdx.x / kw, ke0 = threadIdx.x - kj0 * kw;
   auto load_tile = [&](int kt, int buf) {
     const int kb = kmin + kt * KT, nk = min(KT, kmax + 1 - kb);
     bf16* K = Ks + buf * KT * QS;
     bf16* V = Vs + buf * KT * VS;
-    const int kw = D2 / 8;
-    for (int i = threadIdx.x; i < KT * kw; i += 128) {
-      const int j = i / kw, e = (i - j * kw) * 8;
-      cp_async_16_or_zero(K + j * QS + e, j < nk ? kc + (long long)(kb + j) * NK + e : kc, j < nk);
+    const bf16* ksrc = kc + (long long)kb * NK;
+    const bf16* vsrc = vc + (long long)kb * NV;
+    // rows past the last key are zero, and so are value columns from vdim on; 16-byte chunk (row j, chunk e) by thread, stepping by 128
+#pragma unroll 4
+    for (int j = kj0, e = ke0; j < KT; ) {
+      cp_async_16_or_zero(K + j * QS + e * 8, j < nk ? ksrc + j * NK + e * 8 : kc, j < nk);
+      j += kdj; e += kde;
+      if (e >= kw) { e -= kw; ++j; }
     }
-    for (int i = threadIdx.x; i < KT * VT * 2; i += 128) {      // columns from vdim on, and rows past the last key, are zero
-      const int j = i / (VT * 2), e = (i - j * (VT * 2)) * 8;
+#pragma unroll
+    for (int i = 0; i < KT * VT * 2 / 128; ++i) {
+      const int c = threadIdx.x + i * 128, j = c / (VT * 2), e = (c % (VT * 2)) * 8;
       const bool ok = j < nk && e < vdim;
-      cp_async_16_or_zero(V + j * VS + e, ok ? vc + (long long)(kb + j) * NV + e : vc, ok);
+      cp_async_16_or_zero(V + j * VS + e, ok ? vsrc + j * NV + e : vc, ok);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -414,18 +426,20 @@ __global__ void __launch_bounds__(128, 2) diff_attn_mma_kernel(DiffAttnParams p)
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
         const float mn = fmaxf(rm[m][hf], mx), base = mn > -INFINITY ? mn * L2E : 0.f;
-        const float corr = exp2f(rm[m][hf] * L2E - base);       // 0 before the first visible key
+        const float corr = exp2_approx(rm[m][hf] * L2E - base);       // 0 before the first visible key
         rm[m][hf] = mn;
         float sum = 0.f;
 #pragma unroll
         for (int b = 0; b < 2 * NP; ++b) {
-          const float w0 = exp2f(fmaf(s[b][2 * hf], L2E, -base)), w1 = exp2f(fmaf(s[b][2 * hf + 1], L2E, -base));
+          const float w0 = exp2_approx(fmaf(s[b][2 * hf], L2E, -base)), w1 = exp2_approx(fmaf(s[b][2 * hf + 1], L2E, -base));
           s[b][2 * hf] = w0; s[b][2 * hf + 1] = w1;
           sum += w0 + w1;
         }
         rl[m][hf] = rl[m][hf] * corr + sum;                     // this thread's share of the row's sum
+        if (__any_sync(0xffffffffu, corr != 1.f)) {              // running maxima settle after a few tiles
 #pragma unroll
-        for (int b = 0; b < 2 * VT; ++b) { o[m][b][2 * hf] *= corr; o[m][b][2 * hf + 1] *= corr; }
+          for (int b = 0; b < 2 * VT; ++b) { o[m][b][2 * hf] *= corr; o[m][b][2 * hf + 1] *= corr; }
+        }
       }
 #pragma unroll
       for (int np = 0; np < NP; ++np) {
