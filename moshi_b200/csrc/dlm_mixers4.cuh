@@ -339,7 +339,7 @@ __global__ void __launch_bounds__(128, 2) diff_attn_mma_kernel(DiffAttnParams p)
     // rows past the last key are zero, and so are value columns from vdim on; 16-byte chunk (row j, chunk e) by thread, stepping by 128
 #pragma unroll 4
     for (int j = kj0, e = ke0; j < KT; ) {
-      cp_async_16_or_zero(K + j * QS + e * 8, j < nk ? ksrc + j * NK + e * 8 : kc, j < nk);
+      cp_async_16_or_zero(K + j * QS + e * 8, j < nk ? ksrc + j * (int)NK + e * 8 : kc, j < nk);
       j += kdj; e += kde;
       if (e >= kw) { e -= kw; ++j; }
     }
@@ -347,7 +347,7 @@ __global__ void __launch_bounds__(128, 2) diff_attn_mma_kernel(DiffAttnParams p)
     for (int i = 0; i < KT * VT * 2 / 128; ++i) {
       const int c = threadIdx.x + i * 128, j = c / (VT * 2), e = (c % (VT * 2)) * 8;
       const bool ok = j < nk && e < vdim;
-      cp_async_16_or_zero(V + j * VS + e, ok ? vsrc + j * NV + e : vc, ok);
+      cp_async_16_or_zero(V + j * VS + e, ok ? vsrc + j * (int)NV + e : vc, ok);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
