@@ -30,7 +30,7 @@
 extern "C" {
 #endif
 
-#define B200_ABI_VERSION 7
+#define B200_ABI_VERSION 8
 
 enum {
   B200_OK = 0,
@@ -401,6 +401,23 @@ int b200_frame_read_buffer(b200_frame* f, const char* name, void* dst_dev, int64
  *           router outputs; the choice adds a correction and, with groups > 1, is limited to the groups_keep groups of neighbouring
  *           outputs with the largest single choice score; the `top` best are used with their plain scores as weights; the last
  *           `identity` outputs are experts that return h itself; shared_ff > 0: one more such expert runs for every token
+ * and (the Korirax design):
+ *   block   B200_BLOCK_PARALLEL_RESIDUAL with norm B200_NORM_RMS (a plain weight); side_dim > 0: behind every block
+ *           x += rms(W_proj (gelu_tanh(W_gate x) * e)) * w, e the layer's side_dim elements of the token's row of "side.embed";
+ *           loop_times > 0: layers loop_start .. loop_stop - 1 run loop_times times with the same weights, each pass on a cache and
+ *           state of its own, row t of "loop.step" being added to x in front of pass t
+ *   mixer   B200_MIXER_LATENT_ATTENTION on this block: queries W_uq rms(W_dq h) * w of size q_rank in between, a rotated part as in the
+ *           Dibulix design (adjacent pairs, index ramp), out_gate: the heads' results times sigmoid(W_g h) element by element
+ *           B200_MIXER_BIAS_ATTENTION: causal softmax attention with grouped key/value heads, biased projections, an RMS norm per head
+ *           on q and k (qk_norm), a query factor that grows with the position (q_temp_*), no rotation; the scaled score gets the entry
+ *           of "mix.rel" [B][heads] for the key's distance n: row n below B/2, then a logarithmic scale that reaches the last row at
+ *           bias_max; out_gate as above
+ *           B200_MIXER_RGLRU: y = gelu_tanh(W_y h + b), u = a causal convolution (conv_taps, with a bias) of W_x h + b; gates r, i =
+ *           sigmoid of block-diagonal products of u; log a = -8 r softplus(lam), S <- a S + sqrt(1 - a^2) i u; the result is W_o (S * y)
+ *   mlp     B200_MLP_DENSE_SILU_GLU: W_down (silu(W_gate h) * (W_up h))
+ *           B200_MLP_MOE_GELU: routed experts W_down gelu(W_up h) (the erf form); fp32 scores sigmoid(W_router h), the choice adds a
+ *           correction and, with groups > 1, is limited to the groups_keep groups with the largest sum of two choice scores; the chosen
+ *           scores over their sum, times router_scale, are the weights; shared_ff > 0: one more such expert runs for every token
  * Precision: compute_dtype B200_BF16 = bf16 weights / activations / cache with fp32 accumulation, while norms, attention
  * scores and weights, gates, routers, recurrent state, the residual stream and the depth average stay fp32; B200_F32 =
  * everything in IEEE fp32 (FMA).
@@ -411,10 +428,10 @@ typedef struct b200_dlm b200_dlm;
 
 enum { B200_MIXER_LATENT_ATTENTION = 1, B200_MIXER_WINDOW_ATTENTION = 2, B200_MIXER_GLA = 3, B200_MIXER_MLSTM = 4, B200_MIXER_PARALLEL = 5,
        B200_MIXER_SIGMOID_ATTENTION = 6, B200_MIXER_RETENTION = 7, B200_MIXER_DELTA = 8, B200_MIXER_MINGRU = 9, B200_MIXER_CHANNEL_DELTA = 10,
-       B200_MIXER_DIFF_ATTENTION = 11 };
+       B200_MIXER_DIFF_ATTENTION = 11, B200_MIXER_BIAS_ATTENTION = 12, B200_MIXER_RGLRU = 13 };
 enum { B200_MLP_NONE = 0, B200_MLP_DENSE_RELU2 = 1, B200_MLP_MOE_RELU2 = 2, B200_MLP_DENSE_GATED_GELU = 3, B200_MLP_MOE_CLAMPED_GLU = 4,
-       B200_MLP_DENSE_CLAMPED_GLU = 5, B200_MLP_MOE_SILU_GLU = 6 };
-enum { B200_NORM_RMS_ZERO_CENTRED = 0, B200_NORM_LAYER = 1 };   /* norm of the parallel-residual block */
+       B200_MLP_DENSE_CLAMPED_GLU = 5, B200_MLP_MOE_SILU_GLU = 6, B200_MLP_DENSE_SILU_GLU = 7, B200_MLP_MOE_GELU = 8 };
+enum { B200_NORM_RMS_ZERO_CENTRED = 0, B200_NORM_LAYER = 1, B200_NORM_RMS = 2 };   /* norm of the parallel-residual block */
 enum { B200_BLOCK_GATED_DEPTH_AVERAGE = 0, B200_BLOCK_SANDWICH = 1, B200_BLOCK_PARALLEL_RESIDUAL = 2, B200_BLOCK_PRE_NORM_STREAMS = 3 };
 enum { B200_SINK_LEARNED = 0, B200_SINK_NONE = 1, B200_SINK_UNIT = 2 };   /* what a softmax denominator holds beside the keys */
 #define B200_DLM_MAX_STREAMS 8
@@ -449,6 +466,11 @@ typedef struct {
   int qk_norm;                /* differential attention: RMS norm per head and map on q and k   */
   float diff;                 /* differential attention: lambda's constant; the result is scaled by 1 - diff */
   int kv_from;                /* differential attention: layer whose cached keys and values are read (-1: the layer's own) */
+  int q_rank;                 /* latent attention: size of the queries' latent (0: queries straight from the input) */
+  int out_gate;               /* latent / bias attention: every element of the heads' results times a sigmoid of its own */
+  float bias_max;             /* bias attention: distance from which the last row of the bias table serves */
+  float q_temp_coef, q_temp_every;   /* bias attention: queries times 1 + coef * ln(floor((position + 1) / every) + 1); every <= 0: none */
+  int blocks;                 /* RG-LRU: square gate matrices, each over dim / blocks channels */
 } b200_dlm_mixer;
 
 typedef struct {
@@ -458,11 +480,11 @@ typedef struct {
   int ff;                     /* hidden size of the feed-forward (of one expert)                */
   int experts, top;           /* routed experts and how many of them a token uses               */
   float expert_limit;         /* clamped gated units (experts or dense): bound of the gate (above) and of the value (both sides) */
-  float router_scale;         /* clamped experts: multiplies the normalised weights             */
+  float router_scale;         /* clamped / gelu experts: multiplies the normalised weights             */
   float a_scale, b_scale;     /* pre-norm streams, PARALLEL: the pair's results are summed with these factors */
-  int shared_ff;              /* MOE_SILU_GLU: hidden size of the expert that runs for every token (0: none) */
+  int shared_ff;              /* MOE_SILU_GLU / MOE_GELU: hidden size of the expert that runs for every token (0: none) */
   int identity;               /* MOE_SILU_GLU: router outputs behind the experts that stand for h itself */
-  int groups, groups_keep;    /* MOE_SILU_GLU: equal groups of router outputs, and how many of them a token may choose from (groups <= 1: no limit) */
+  int groups, groups_keep;    /* MOE_SILU_GLU / MOE_GELU: equal groups of router outputs, and how many of them a token may choose from (groups <= 1: no limit) */
 } b200_dlm_layer;
 
 typedef struct {
@@ -477,6 +499,8 @@ typedef struct {
   float logit_scale;          /* pre-norm streams: multiplies the logits                         */
   int tied_head;              /* the logits come from the embedding table (no "head" tensor)     */
   int norm;                   /* parallel residual: B200_NORM_*                                  */
+  int side_dim;               /* parallel residual: size of the per-layer token input (0: none)  */
+  int loop_start, loop_stop, loop_times;   /* parallel residual: layers loop_start .. loop_stop - 1 run loop_times times in a row (0: no loop) */
 } b200_dlm_config;
 
 int b200_dlm_create(const b200_dlm_config* cfg, b200_dlm** out);
@@ -515,8 +539,8 @@ int b200_dlm_step(b200_dlm* h, int n_entries, const int32_t* slots_host, const i
 /* One token per logit row of the last step.  use_sampling = 0 or temp <= 0: the first maximum of the fp32 logits.  Otherwise the
  * LM's sampler (b200_op_sample) on their bf16 rounding: noise f32 [n_want][min(top_k, vocab)] Exp(1) draws. */
 int b200_dlm_sample(b200_dlm* h, const float* noise_dev, int use_sampling, float temp, int top_k, int64_t* out_dev);
-/* Debug / test hand-offs of the last step, copied device-to-device: "layers" f32 [n_layers][tokens][width] (needs option
- * trace_layers = 1: what each layer hands on), "logits" f32 [n_want][vocab]. */
+/* Debug / test hand-offs of the last step, copied device-to-device: "layers" f32 [layer runs][tokens][width] (needs
+ * option trace_layers = 1: what each layer hands on, once per pass of a loop), "logits" f32 [n_want][vocab]. */
 int b200_dlm_read_buffer(b200_dlm* h, const char* name, void* dst_dev, int64_t capacity_bytes, int64_t* nbytes);
 /* HBM bytes one step must move / FLOPs it must do for `tokens` new tokens on top of `context` cached ones (roofline of bench.py) */
 int64_t b200_dlm_algorithmic_bytes(b200_dlm* h, int tokens, int context);

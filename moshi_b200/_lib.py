@@ -14,7 +14,7 @@ LIB_PATH = Path(__file__).resolve().parent / "_C" / "libmoshi_b200.so"
 
 B200_OK, B200_ERR_INVALID, B200_ERR_SHAPE, B200_ERR_STATE, B200_ERR_CUDA, B200_ERR_MISSING = range(6)
 B200_F32, B200_BF16, B200_F16, B200_I64, B200_U8, B200_I8 = range(6)
-ABI_VERSION = 7
+ABI_VERSION = 8
 
 
 class MimiConfigC(C.Structure):
@@ -48,7 +48,8 @@ class DLMMixerC(C.Structure):
                 ("gate_cap", C.c_float), ("tau", C.c_float), ("rot_pairing", C.c_int), ("rot_scaling", C.c_int), ("rot_fast", C.c_float),
                 ("rot_slow", C.c_float), ("softcap", C.c_float), ("v_mix", C.c_int), ("decay", C.POINTER(C.c_float)),
                 ("bias", C.c_int), ("sink", C.c_int), ("head_gate", C.c_int), ("chunk", C.c_int), ("qk_norm", C.c_int), ("diff", C.c_float),
-                ("kv_from", C.c_int)]
+                ("kv_from", C.c_int), ("q_rank", C.c_int), ("out_gate", C.c_int), ("bias_max", C.c_float), ("q_temp_coef", C.c_float),
+                ("q_temp_every", C.c_float), ("blocks", C.c_int)]
 
 
 class DLMLayerC(C.Structure):
@@ -61,7 +62,8 @@ class DLMConfigC(C.Structure):
     _fields_ = [("vocab", C.c_int), ("width", C.c_int), ("n_layers", C.c_int), ("embedding_scale", C.c_float),
                 ("residual_mult", C.c_float), ("norm_eps", C.c_float), ("compute_dtype", C.c_int), ("block", C.c_int),
                 ("canon_taps", C.c_int), ("logit_softcap", C.c_float), ("layers", C.POINTER(DLMLayerC)),
-                ("streams", C.c_int), ("logit_scale", C.c_float), ("tied_head", C.c_int), ("norm", C.c_int)]
+                ("streams", C.c_int), ("logit_scale", C.c_float), ("tied_head", C.c_int), ("norm", C.c_int),
+                ("side_dim", C.c_int), ("loop_start", C.c_int), ("loop_stop", C.c_int), ("loop_times", C.c_int)]
 
 
 _P = C.c_void_p

@@ -271,17 +271,18 @@ def tiny_lm_config(**over) -> LMConfig:
 # ---------------------------------------------------------------------------------------------------
 MIXERS = {"latent_attention": 1, "window_attention": 2, "gla": 3, "mlstm": 4, "parallel": 5,    # name -> B200_MIXER_*
           "sigmoid_attention": 6, "retention": 7, "delta": 8, "mingru": 9, "channel_delta": 10,
-          "diff_attention": 11}
+          "diff_attention": 11, "bias_attention": 12, "rglru": 13}
 # feed-forward kind -> B200_MLP_*: "dense" / "moe" are the squared-ReLU layers (a null "mlp" = none), "gated_gelu" a gated dense
 # layer with the tanh form of GELU, "moe_clamped_glu" routed experts with clamped gates behind a sigmoid router, "clamped_glu" such
-# a gated unit alone, "moe_silu_glu" routed experts with silu gates behind a softmax router (groups, identity and shared experts)
-MLP_KINDS = {None: 0, "dense": 1, "moe": 2, "gated_gelu": 3, "moe_clamped_glu": 4, "clamped_glu": 5, "moe_silu_glu": 6}
+# a gated unit alone, "moe_silu_glu" routed experts with silu gates behind a softmax router (groups, identity and shared experts),
+# "silu_glu" a dense layer with a silu gate, "moe_gelu" routed experts without a gate (erf GELU) behind a sigmoid router (groups, shared)
+MLP_KINDS = {None: 0, "dense": 1, "moe": 2, "gated_gelu": 3, "moe_clamped_glu": 4, "clamped_glu": 5, "moe_silu_glu": 6, "silu_glu": 7, "moe_gelu": 8}
 BLOCKS = {"gated_depth_average": 0, "sandwich": 1, "parallel_residual": 2, "pre_norm_streams": 3}  # block arrangement -> B200_BLOCK_*
 NO_WINDOW = 1 << 30                                                                               # a window attention without a mask: every earlier key is seen
 SINKS = {"learned": 0, "none": 1, "unit": 2}                                                      # softmax denominator's extra term -> B200_SINK_*
 ROT_PAIRINGS = {"halves": 0, "adjacent": 1}                                                       # -> B200_ROT_HALVES / B200_ROT_ADJACENT
 ROT_SCALINGS = {None: 0, "bands": 1, "ramp": 2, "linear": 3}                                      # -> B200_ROT_PLAIN / BANDS / RAMP / LINEAR
-NORMS = {"rms_zero_centred": 0, "layer": 1}                                                       # norm of the parallel-residual block -> B200_NORM_*
+NORMS = {"rms_zero_centred": 0, "layer": 1, "rms": 2}                                             # norm of the parallel-residual block -> B200_NORM_*
 
 
 @dataclass
@@ -305,7 +306,12 @@ class MixerConfig:
     query / key dimensions per head beside its ``dim`` unrotated ones; the rotated key part is one row shared by the heads.
     ``diff_attention``: two query / key maps per head over the same values, combined as a1 - lambda a2 (``diff`` is lambda's
     constant), keys of the query's own ``chunk`` of positions (0: all earlier ones), ``qk_norm`` an RMS norm per head and map,
-    ``kv_from`` the layer whose cached keys and values are read (-1: its own); ``rot_scaling_kind`` "linear" reads {factor}."""
+    ``kv_from`` the layer whose cached keys and values are read (-1: its own); ``rot_scaling_kind`` "linear" reads {factor}.
+    ``bias_attention``: softmax attention without rotation, a learned bias per head and distance bucket added to the scores
+    (``bias_max``: the distance from which the last bucket serves; ``bias_buckets`` is a tensor's shape, not a config key), queries times
+    1 + ``q_temp_coef`` ln(floor((position + 1) / ``q_temp_every``) + 1).  ``q_rank``: a latent attention's queries come through a
+    normed latent of that size.  ``out_gate``: every element of the heads' results times a sigmoid of its own.  ``rglru``: a gated
+    linear recurrence of ``dim`` channels behind a convolution of ``conv`` taps, its gates from ``blocks`` square matrices."""
     kind: str
     heads: int
     dim: int
@@ -334,6 +340,13 @@ class MixerConfig:
     qk_norm: bool = False
     diff: float = 0.0
     kv_from: int = -1
+    q_rank: int = 0
+    out_gate: bool = False
+    bias_max: float = 0.0
+    bias_buckets: int = 32
+    q_temp_coef: float = 0.0
+    q_temp_every: float = 0.0
+    blocks: int = 0
 
 
 def _window_attention_from_dict(m: dict) -> MixerConfig:
@@ -446,6 +459,10 @@ class DecoderLMConfig:
     logit_scale: float = 1.0
     tied_head: bool = False             # the logits come from the embedding table
     norm: str = "rms_zero_centred"      # parallel_residual: the block's norm
+    side_dim: int = 0                   # parallel_residual: size of the token's second embedding that every layer adds through a gate (0: none)
+    loop_start: int = 0                 # parallel_residual: layers loop_start .. loop_stop - 1 run loop_times times in a row with the same
+    loop_stop: int = 0                  # weights, every pass on caches of its own and with a vector of its own added in front
+    loop_times: int = 0                 # (0: no loop)
 
     @staticmethod
     def from_dict(d: dict) -> "DecoderLMConfig":
@@ -458,6 +475,13 @@ class DecoderLMConfig:
                                layers=[DecoderLayerConfig.from_dict(x) for x in d["layers"]],
                                embedding_scale=float(d["embedding"]["scale"]), residual_mult=float(d["residual_mult"]),
                                norm_eps=float(d["norm"]["eps"]))
+
+    def layer_runs(self) -> tp.List[int]:
+        """The layers in the order a token runs through them."""
+        n = len(self.layers)
+        if not self.loop_times:
+            return list(range(n))
+        return list(range(self.loop_start)) + list(range(self.loop_start, self.loop_stop)) * self.loop_times + list(range(self.loop_stop, n))
 
     @staticmethod
     def from_json(path: str) -> "DecoderLMConfig":
@@ -865,6 +889,138 @@ class MegolornConfig(DecoderLMConfig):
         return out
 
 
+@dataclass
+class KoriraxConfig(DecoderLMConfig):
+    """``config.json`` of the Korirax design: parallel blocks (one RMS norm feeds mixer and feed-forward, ``x += mixer(h) + ff(h)``)
+    with a per-layer token input behind them, a scaled embedding, and a stretch of layers that runs several times (``loop``).  Layers
+    are ``latent_attention`` (queries through a latent too, a rotated key part shared by the heads, adjacent pairs with the index
+    ramp), ``attention`` (biased projections, a norm per head on queries and keys, no rotation, a bias by distance, queries that grow
+    with the position), both with a gate per element, or ``rglru`` (a gated linear recurrence behind a short convolution), each with a
+    ``dense`` (silu-gated) or ``moe`` (sigmoid router with a choice correction and groups, erf-GELU experts, a shared expert)
+    feed-forward or none."""
+
+    TYPES = {"latent_attention": "latent_attention", "attention": "bias_attention", "rglru": "rglru"}
+
+    @staticmethod
+    def _layer(i: int, d: dict) -> DecoderLayerConfig:
+        t, m, mlp = d["type"], d["mixer"], d.get("mlp")
+        if t not in KoriraxConfig.TYPES:
+            raise ValueError(f"layer {i}: a Korirax layer is one of {sorted(KoriraxConfig.TYPES)}, not {t!r}")
+        kind = KoriraxConfig.TYPES[t]
+        if t == "latent_attention":
+            rot, rd = dict(m.get("rot") or {}), int(m.get("rot_dim", 0))
+            if rd and int(rot.get("dims", rd)) != rd:
+                raise ValueError(f"layer {i}: the rotation covers the rotated part (rot.dims = rot_dim)")
+            rot["dims"] = rd
+            a = MixerConfig(kind=kind, heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]), q_rank=int(m["q_rank"]),
+                            scale=float(m["scale"]), sink="none", out_gate=True, **_rot_fields({"rot": rot}, "adjacent"))
+        elif t == "attention":
+            qt = m.get("q_temp") or {}
+            a = MixerConfig(kind=kind, heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
+                            sink="none", bias=True, qk_norm=True, out_gate=True, bias_max=float(m["bias_max"]), bias_buckets=int(m.get("bias_buckets", 32)),
+                            q_temp_coef=float(qt.get("coef", 0.0)), q_temp_every=float(qt.get("every", 0.0)))
+        else:
+            a = MixerConfig(kind=kind, heads=1, dim=int(m["width"]), vdim=int(m["width"]), conv=int(m["conv"]), blocks=int(m["blocks"]), bias=True)
+            if a.blocks < 1 or a.dim % a.blocks:
+                raise ValueError(f"layer {i}: blocks must cut the recurrence's width into equal parts")
+        if mlp is None:
+            return DecoderLayerConfig(type=kind, mlp_kind=None, a=a)
+        if mlp["kind"] == "dense":
+            return DecoderLayerConfig(type=kind, mlp_kind="silu_glu", ff=int(mlp["ff"]), a=a)
+        if mlp["kind"] != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        r, g, sh = mlp["router"], mlp["router"].get("groups") or {}, mlp.get("shared") or {}
+        return DecoderLayerConfig(type=kind, mlp_kind="moe_gelu", ff=int(mlp["expert"]["ff"]), a=a, experts=int(r["experts"]), top=int(r["top"]),
+                                  router_scale=float(r.get("scale", 1.0)), groups=int(g.get("count", 1)), groups_keep=int(g.get("keep", 1)),
+                                  shared_ff=int(sh.get("ff", 0)))
+
+    @staticmethod
+    def from_dict(d: dict) -> "KoriraxConfig":
+        loop, n = d.get("loop") or {}, len(d["layers"])
+        start, stop, times = int(loop.get("start", 0)), int(loop.get("stop", 0)), int(loop.get("times", 0))
+        if loop and not (0 <= start < stop <= n and times >= 1):
+            raise ValueError(f"loop: layers {start} .. {stop - 1} x {times} is not a stretch of the {n} layers")
+        return KoriraxConfig(architecture=d["architecture"], vocab=int(d["vocab"]), width=int(d["width"]),
+                             layers=[KoriraxConfig._layer(i, x) for i, x in enumerate(d["layers"])],
+                             embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)), norm_eps=float(d["norm"]["eps"]),
+                             block="parallel_residual", norm="rms", side_dim=int((d.get("token_side") or {}).get("dim", 0)),
+                             loop_start=start, loop_stop=stop, loop_times=times)
+
+    @staticmethod
+    def _layer_to_dict(L: DecoderLayerConfig) -> dict:
+        a = L.a
+        if a.kind == "latent_attention":
+            mixer: dict = {"dim": a.dim, "heads": a.heads, "kv_rank": a.kv_rank, "q_rank": a.q_rank, "rot_dim": a.rot_dims, "scale": a.scale, "vdim": a.vdim}
+            rot = _rot_to_dict(a)
+            if rot is not None:
+                mixer["rot"] = rot
+            t = "latent_attention"
+        elif a.kind == "bias_attention":
+            mixer, t = {"bias_max": a.bias_max, "dim": a.dim, "heads": a.heads, "kv_heads": a.kv_heads, "scale": a.scale, "vdim": a.vdim}, "attention"
+            if a.q_temp_every:
+                mixer["q_temp"] = {"coef": a.q_temp_coef, "every": a.q_temp_every}
+        else:
+            mixer, t = {"blocks": a.blocks, "conv": a.conv, "width": a.dim}, "rglru"
+        if L.mlp_kind is None:
+            mlp = None
+        elif L.mlp_kind == "silu_glu":
+            mlp = {"ff": L.ff, "kind": "dense"}
+        else:
+            router: dict = {"experts": L.experts, "scale": L.router_scale, "top": L.top}
+            if L.groups > 1:
+                router["groups"] = {"count": L.groups, "keep": L.groups_keep}
+            mlp = {"expert": {"ff": L.ff}, "kind": "moe", "router": router}
+            if L.shared_ff:
+                mlp["shared"] = {"ff": L.shared_ff}
+        return {"mixer": mixer, "mlp": mlp, "type": t}
+
+    def to_dict(self) -> dict:
+        d: dict = {"architecture": self.architecture, "embedding": {"scale": self.embedding_scale},
+                   "layers": [self._layer_to_dict(x) for x in self.layers], "norm": {"eps": self.norm_eps}, "vocab": self.vocab, "width": self.width}
+        if self.loop_times:
+            d["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
+        if self.side_dim:
+            d["token_side"] = {"dim": self.side_dim}
+        return d
+
+    def tensor_shapes(self) -> dict:
+        W, D = self.width, self.side_dim
+        out: dict = {"embed": (self.vocab, W)}
+        if self.loop_times:
+            out["loop.step"] = (self.loop_times, W)
+        if D:
+            out["side.embed"] = (self.vocab, len(self.layers) * D)
+        for i, L in enumerate(self.layers):
+            p, m, a = f"l{i}.", f"l{i}.mix.", L.a
+            out[p + "norm1"] = (W,)
+            Kv = a.heads * a.vdim
+            if a.kind == "latent_attention":
+                out.update({m + "dq": (a.q_rank, W), m + "dq.norm": (a.q_rank,), m + "uq": (a.heads * (a.dim + a.rot_dims), a.q_rank),
+                            m + "dkv": (a.kv_rank + a.rot_dims, W), m + "dkv.norm": (a.kv_rank,), m + "uk": (a.heads * a.dim, a.kv_rank),
+                            m + "uv": (Kv, a.kv_rank), m + "g": (Kv, W), m + "o": (W, Kv)})
+            elif a.kind == "bias_attention":
+                for nm, rows in (("q", a.heads * a.dim), ("k", a.kv_heads * a.dim), ("v", a.kv_heads * a.vdim)):
+                    out.update({m + nm: (rows, W), m + nm + ".b": (rows,)})
+                out.update({m + "q.norm": (a.dim,), m + "k.norm": (a.dim,), m + "rel": (a.bias_buckets, a.heads), m + "g": (Kv, W), m + "o": (W, Kv)})
+            else:
+                n, nb = a.dim, a.blocks
+                out.update({m + "y": (n, W), m + "y.b": (n,), m + "x": (n, W), m + "x.b": (n,), m + "conv": (n, a.conv), m + "conv.b": (n,),
+                            m + "ra": (nb, n // nb, n // nb), m + "ra.b": (nb, n // nb), m + "ri": (nb, n // nb, n // nb), m + "ri.b": (nb, n // nb),
+                            m + "lam": (n,), m + "o": (W, n)})
+            if L.mlp_kind == "silu_glu":
+                out.update({p + "mlp.gate": (L.ff, W), p + "mlp.up": (L.ff, W), p + "mlp.down": (W, L.ff)})
+            elif L.mlp_kind == "moe_gelu":
+                for e in range(L.experts):
+                    out.update({p + f"mlp.e{e}.up": (L.ff, W), p + f"mlp.e{e}.down": (W, L.ff)})
+                out.update({p + "mlp.router": (L.experts, W), p + "mlp.correction": (L.experts,)})
+                if L.shared_ff:
+                    out.update({p + "mlp.shared.up": (L.shared_ff, W), p + "mlp.shared.down": (W, L.shared_ff)})
+            if D:
+                out.update({p + "side.gate": (D, W), p + "side.proj": (W, D), p + "side.norm": (W,)})
+        out.update({"final.norm": (W,), "head": (self.vocab, W)})
+        return out
+
+
 # architecture name in config.json -> configuration class (the model registry of the text-only decoder LMs)
 DECODER_ARCHITECTURES: dict = {"Likosun": DecoderLMConfig, "Govuvik": GovuvikConfig, "Namalix": NamalixConfig, "Dibulix": DibulixConfig,
-                               "Megolorn": MegolornConfig}
+                               "Megolorn": MegolornConfig, "Korirax": KoriraxConfig}

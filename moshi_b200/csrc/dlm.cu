@@ -3,8 +3,9 @@
 // state of recurrent mixers), and the ragged step (any number of new tokens per slot) that both prompt portions and
 // single-token decoding go through.  Block arrangements: gated parallel sublayers with a depth-weighted
 // average (the Likosun design), RMS-norm sandwiches around mixer and feed-forward in turn (the Govuvik design), a plain parallel
-// block on one zero-centred RMS norm (the Namalix design) or one layer norm (the Megolorn design), and pre-norm sublayers on
-// residual streams (the Dibulix design).
+// block on one zero-centred RMS norm (the Namalix design), one layer norm (the Megolorn design) or one RMS norm with a per-layer token
+// input and a stretch of layers that runs several times (the Korirax design), and pre-norm sublayers on residual streams (the Dibulix
+// design).
 #include <algorithm>
 
 #include <cmath>
@@ -14,6 +15,7 @@
 #include "dlm_mixers2.cuh"
 #include "dlm_mixers3.cuh"
 #include "dlm_mixers4.cuh"
+#include "dlm_mixers5.cuh"
 #include "gemm_sk.cuh"
 #include "lm_kernels.cuh"
 
@@ -79,6 +81,19 @@ struct Layer {
   int kv_src = -1, rot_id = -1, glu_ff = 0, ob_ld = 0, ob_act = 0, mma_vt = 0;
   size_t smem_mma_one = 0;
   float lambda = 0.f;
+  // ---- joint layers of the parallel-residual block (finalize_joint_layer): as above one projection and one output product.  Latent
+  // attention [dq | dkv | g | ..] with the queries' second product `uq`; bias attention [q | k | v | g | ..]; RG-LRU [y | x | ..]
+  Weight uq, side_gate, side_proj;
+  void* side_gate_rm = nullptr;        // T [side_dim][width], row-major (the few-token kernel)
+  float *side_norm = nullptr, *rel = nullptr;      // rel: [heads][far + 1] biases over distances
+  int far = 0, far_smem = 0;
+  float *conv_b = nullptr, *x_b = nullptr, *y_b = nullptr, *gate_b = nullptr, *lam8 = nullptr;
+  void* gates = nullptr;               // T [blocks][2 bs][bs]
+  // ---- layer runs: with a loop the handle's list holds a copy of a layer per pass, which shares the weights and owns its cache
+  int index = 0;                       // the layer's number in the configuration
+  const float* step = nullptr;         // vector added to the residual in front of this run (first layer of a pass)
+  bool repeat = false;                 // not the first run of its layer
+  int64_t wbytes = 0;
 };
 
 // attention tile list of one (heads, rows per tile) combination
@@ -142,9 +157,12 @@ struct b200_dlm {
   int vmix_first = -1;                 // the first attention layer that blends values: the later ones blend its values in
   float* small32 = nullptr;            // [tokens][nsmall] fp32 results of the small projection
   float* xs = nullptr;                 // pre-norm streams block: the residual streams [tokens][streams][width]
+  float* loop_step = nullptr;          // [loop_times][width]
+  void *side_embed = nullptr, *sidez = nullptr, *cq = nullptr, *q2 = nullptr;      // T [vocab][n_layers * side_dim]; step buffers: side product, query latents, queries
+  int side_ld = 0, side_cols = 0;
   float *rows3 = nullptr, *gend = nullptr;      // chunked delta rule with a decay per key channel: [tokens][heads][3 dim], [chunks][heads][dim]
-  struct Rotation { b200_dlm_mixer m; double* freq; float* table; };
-  std::vector<Rotation> rots;          // distinct rotations of the differential attention layers; table: [tokens][rot_dims], filled once per step
+  struct Rotation { b200_dlm_mixer m; double* freq; float amp; float* table; };
+  std::vector<Rotation> rots;          // distinct rotations of the layers that read them from a table; table: [tokens][rot_dims], filled once per step
   void *vfirst = nullptr, *act2 = nullptr;      // T [tokens][G * vdim] values of layer vmix_first; T [tokens * top][2 ff] experts' first product
 };
 
@@ -207,26 +225,26 @@ int seal_weight(b200_dlm* h, Weight& w, void* rm, int N, int K, std::vector<void
 template <typename TA, typename TB, typename TC>
 int gemm_nt(cudaStream_t st, const TA* A, long long lda, long long sa, const TB* B, long long ldb, long long sb, TC* C, long long ldc,
             long long sc, int M, int N, int K, int batch, float alpha, int accumulate = 0, int outer = 1, long long sa2 = 0, long long sb2 = 0,
-            long long sc2 = 0) {
+            long long sc2 = 0, const TC* gate = nullptr, long long ldg = 0, long long sg = 0) {
   dim3 grid(ceil_div(N, 64), ceil_div(M, 64), batch * outer);
-  B200_LAUNCH((gemm_nt_kernel<TA, TB, TC>), grid, 256, 0, st, A, lda, sa, B, ldb, sb, C, ldc, sc, M, N, K, alpha, accumulate, outer > 1 ? batch : 0, sa2, sb2, sc2);
+  B200_LAUNCH((gemm_nt_kernel<TA, TB, TC>), grid, 256, 0, st, A, lda, sa, B, ldb, sb, C, ldc, sc, M, N, K, alpha, accumulate, outer > 1 ? batch : 0, sa2, sb2, sc2, gate, ldg, sg);
   return check_launch("gemm_nt");
 }
 
 // the per-head products around the latent attention: tensor cores for bf16 weights (K a multiple of 16), else CUDA cores
 template <typename TA, typename TB, typename TC>
 int head_gemm(cudaStream_t st, const TA* A, long long lda, long long sa, const TB* B, long long ldb, long long sb, TC* C, long long ldc,
-              long long sc, int M, int N, int K, int batch, float alpha, bool tensor_cores) {
+              long long sc, int M, int N, int K, int batch, float alpha, bool tensor_cores, const TC* gate = nullptr, long long ldg = 0, long long sg = 0) {
   if constexpr (sizeof(TB) == 2) {
     constexpr long long AE = 16 / (long long)sizeof(TA);       // elements of A per 16 bytes
     const bool aligned = lda % AE == 0 && sa % AE == 0 && ldb % 8 == 0 && sb % 8 == 0 && (uintptr_t)A % 16 == 0 && (uintptr_t)B % 16 == 0;
     if (tensor_cores && K % 16 == 0 && aligned) {
       dim3 grid(ceil_div(N, 64), ceil_div(M, 64), batch);
-      B200_LAUNCH((gemm_nt_mma_kernel<TA, TC>), grid, 128, 0, st, A, lda, sa, B, ldb, sb, C, ldc, sc, M, N, K, alpha);
+      B200_LAUNCH((gemm_nt_mma_kernel<TA, TC>), grid, 128, 0, st, A, lda, sa, B, ldb, sb, C, ldc, sc, M, N, K, alpha, gate, ldg, sg);
       return check_launch("gemm_nt_mma");
     }
   }
-  return gemm_nt(st, A, lda, sa, B, ldb, sb, C, ldc, sc, M, N, K, batch, alpha);
+  return gemm_nt(st, A, lda, sa, B, ldb, sb, C, ldc, sc, M, N, K, batch, alpha, 0, 1, 0, 0, 0, gate, ldg, sg);
 }
 
 // y[M][N] = x[M][K] . W^T in the compute type
@@ -1020,6 +1038,73 @@ int put_glu_experts(b200_dlm* h, Layer& L, const std::string& p) {
   return B200_OK;
 }
 
+// the rotation's entry in the handle's list; layers with the same rotation share its table
+int add_rotation(b200_dlm* h, const b200_dlm_mixer& a, int* id) {
+  *id = -1;
+  if (a.rot_dims <= 0) return B200_OK;
+  for (size_t k = 0; k < h->rots.size() && *id < 0; ++k) {
+    const b200_dlm_mixer& r = h->rots[k].m;
+    if (r.rot_dims == a.rot_dims && r.rot_base == a.rot_base && r.rot_scaling == a.rot_scaling && r.rot_factor == a.rot_factor &&
+        (a.rot_scaling != B200_ROT_RAMP || (r.rot_original == a.rot_original && r.rot_fast == a.rot_fast && r.rot_slow == a.rot_slow))) *id = (int)k;
+  }
+  if (*id >= 0) return B200_OK;
+  b200_dlm::Rotation r{a, nullptr, 1.f, nullptr};
+  const std::vector<double> fr = a.rot_scaling == B200_ROT_RAMP ? rotary_frequencies_ramp(a, &r.amp) : rotary_frequencies(a);
+  B200_TRY(h->weights.alloc_t(&r.freq, fr.size(), false));
+  B200_CUDA(cudaMemcpy(r.freq, fr.data(), fr.size() * sizeof(double), cudaMemcpyHostToDevice));
+  h->rots.push_back(r);
+  *id = (int)h->rots.size() - 1;
+  return B200_OK;
+}
+
+// the output products of a mixer and of the gated unit beside it as one: [o | down] against rows [heads' results | unit]
+int put_joint_output(b200_dlm* h, Layer& L, const std::string& o, const std::string& down, int Kv, std::vector<void*>& drop) {
+  const int64_t W = h->cfg.width;
+  const size_t es = esize(h);
+  auto pad8 = [](int v) { return (v + 7) / 8 * 8; };
+  L.ob_act = pad8(Kv); L.ob_ld = L.glu_ff ? pad8(L.ob_act + L.glu_ff) : pad8(Kv);
+  void *wo = nullptr, *tmp = nullptr;
+  B200_TRY(h->weights.alloc(&wo, (size_t)W * L.ob_ld * es, true));
+  B200_CUDA(cudaMalloc(&tmp, (size_t)W * std::max(Kv, L.glu_ff) * es));
+  auto place = [&](const std::string& name, int K, int off) -> int {
+    B200_TRY(put_matrix(h, name, W, K, tmp));
+    B200_CUDA(cudaMemcpy2D(static_cast<char*>(wo) + (size_t)off * es, (size_t)L.ob_ld * es, tmp, (size_t)K * es, (size_t)K * es, (size_t)W, cudaMemcpyDeviceToDevice));
+    return B200_OK;
+  };
+  int rc = place(o, Kv, 0);
+  if (rc == B200_OK && L.glu_ff) rc = place(down, L.glu_ff, L.ob_act);
+  cudaDeviceSynchronize();
+  cudaFree(tmp);
+  B200_TRY(rc);
+  return seal_weight(h, L.o, wo, (int)W, L.ob_ld, drop, (int)W);
+}
+
+// tiles of the one- and two-map attention kernels; rows are (token, query head of one key/value head)
+int plan_map_attention(b200_dlm* h, Layer& L, int i, int nm) {
+  const b200_dlm_mixer& a = L.c.a;
+  const int rep = a.heads / a.kv_heads;
+  L.QT = 0;
+  for (int kt : {32, 16, 8})
+    for (int mr : {8, 4, 1}) {
+      const size_t sm = map_attn_smem(nm, a.dim, a.vdim, mr, kt);
+      if (!L.QT && sm <= 200 * 1024) { L.QT = mr; L.KT = kt; L.attn_smem = sm; }
+    }
+  if (!L.QT) B200_FAIL(B200_ERR_SHAPE, "decoder LM: layer %d: the attention's heads do not fit shared memory", i);
+  L.sig = add_sig(h, rep, L.QT);
+  if (!h->f32 && a.dim % 16 == 0 && a.vdim % 16 == 0 && a.vdim <= 256 / nm) {
+    L.mma_vt = ceil_div(a.vdim, 32) * 2;
+    if (L.mma_vt > 8) L.mma_vt = L.mma_vt <= 12 ? 12 : 16;
+    L.mma_smem = map_attn_mma_smem(nm, a.dim, L.mma_vt, false);
+    L.smem_mma_one = map_attn_mma_smem(nm, a.dim, L.mma_vt, true);
+    // the bias rows of one key/value head: a copy in shared memory where it costs little
+    const size_t rows = L.rel ? (size_t)rep * (L.far + 1) * 4 : 0;
+    L.far_smem = rows > 0 && rows <= 24 * 1024;
+    if (L.far_smem) { L.mma_smem += rows; L.smem_mma_one += rows; }
+    if (std::max(L.mma_smem, L.smem_mma_one) <= 220 * 1024) { L.sig_mma = add_sig(h, rep, 64); L.sig_one = add_sig(h, rep, 16); }
+  }
+  return B200_OK;
+}
+
 // a layer of the parallel-residual block with differential attention (its norm is loaded already)
 int finalize_diff_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
   Layer& L = h->layers[i];
@@ -1082,20 +1167,7 @@ int finalize_diff_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
     }
     L.lambda = (float)(std::exp(dot[0]) - std::exp(dot[1]) + a.diff);
   }
-  if (a.rot_dims > 0) {      // layers with the same rotation share its table
-    for (size_t k = 0; k < h->rots.size() && L.rot_id < 0; ++k) {
-      const b200_dlm_mixer& r = h->rots[k].m;
-      if (r.rot_dims == a.rot_dims && r.rot_base == a.rot_base && r.rot_scaling == a.rot_scaling && r.rot_factor == a.rot_factor) L.rot_id = (int)k;
-    }
-    if (L.rot_id < 0) {
-      b200_dlm::Rotation r{a, nullptr, nullptr};
-      const std::vector<double> fr = rotary_frequencies(a);
-      B200_TRY(h->weights.alloc_t(&r.freq, fr.size(), false));
-      B200_CUDA(cudaMemcpy(r.freq, fr.data(), fr.size() * sizeof(double), cudaMemcpyHostToDevice));
-      h->rots.push_back(r);
-      L.rot_id = (int)h->rots.size() - 1;
-    }
-  }
+  B200_TRY(add_rotation(h, a, &L.rot_id));
   // the small fp32 projection: head gates | router logits
   const int n_route = moe ? L.c.experts + L.c.identity : 0;
   L.s_gate = 0; L.s_router = a.head_gate ? H : 0; L.nsmall = L.s_router + n_route;
@@ -1106,41 +1178,221 @@ int finalize_diff_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
     if (moe) B200_TRY(put_matrix(h, p + "mlp.router", n_route, W, sat(L.s_router)));
     h->weight_bytes += (int64_t)L.nsmall * W * es;
   }
-  // both sublayers' output products as one: [o | down] against rows [heads' results | gated unit]
-  const int Kv = H * a.vdim;
-  L.ob_act = pad8(Kv); L.ob_ld = L.glu_ff ? pad8(L.ob_act + L.glu_ff) : Kv;
-  void *wo = nullptr, *tmp = nullptr;
-  B200_TRY(h->weights.alloc(&wo, (size_t)W * L.ob_ld * es, true));
-  B200_CUDA(cudaMalloc(&tmp, (size_t)W * std::max(Kv, L.glu_ff) * es));
-  int rc = put_matrix(h, m + "o", W, Kv, tmp);
-  if (rc == B200_OK && cudaMemcpy2D(wo, (size_t)L.ob_ld * es, tmp, (size_t)Kv * es, (size_t)Kv * es, (size_t)W, cudaMemcpyDeviceToDevice) != cudaSuccess) rc = B200_ERR_CUDA;
-  if (rc == B200_OK && L.glu_ff) {
-    rc = put_matrix(h, glu + "down", W, L.glu_ff, tmp);
-    if (rc == B200_OK && cudaMemcpy2D(static_cast<char*>(wo) + (size_t)L.ob_act * es, (size_t)L.ob_ld * es, tmp, (size_t)L.glu_ff * es, (size_t)L.glu_ff * es, (size_t)W, cudaMemcpyDeviceToDevice) != cudaSuccess) rc = B200_ERR_CUDA;
-  }
-  cudaDeviceSynchronize();
-  cudaFree(tmp);
-  B200_TRY(rc);
-  B200_TRY(seal_weight(h, L.o, wo, (int)W, L.ob_ld, drop, (int)W));
+  B200_TRY(put_joint_output(h, L, m + "o", glu + "down", H * a.vdim, drop));
   if (moe) {
     B200_TRY(get_f32(h, p + "mlp.correction", n_route, &L.correction));
     B200_TRY(put_glu_experts(h, L, p));
   }
-  // kernels: rows are (token, query head of one key/value head)
-  const int rep = H / G;
-  L.QT = 0;
-  for (int kt : {32, 16, 8})
-    for (int mr : {8, 4, 1}) {
-      const size_t sm = diff_attn_smem(a.dim, a.vdim, mr, kt);
-      if (!L.QT && sm <= 200 * 1024) { L.QT = mr; L.KT = kt; L.attn_smem = sm; }
+  return plan_map_attention(h, L, i, 2);
+}
+
+__global__ void interleave_pairs_kernel(const float* __restrict__ a, const float* __restrict__ b, float* __restrict__ out, int n) {
+  const int i = blockIdx.x * 256 + threadIdx.x;
+  if (i < n) { out[2 * i] = a[i]; out[2 * i + 1] = b[i]; }
+}
+
+// the bias table [B][heads] over distance buckets -> [heads][far + 1] over distances; from `far` on every distance has the last bucket.
+// Bucket of distance n: n below B / 2, then B / 2 + floor(ln(n / (B / 2)) / ln(bias_max / (B / 2)) * (B - B / 2)), at most B - 1.
+int put_distance_bias(b200_dlm* h, const std::string& name, Layer& L, int i) {
+  const b200_dlm_mixer& a = L.c.a;
+  const Tensor* t = h->store.find(name);
+  if (!t || t->shape.size() != 2 || t->shape[1] != a.heads || t->shape[0] < 2) B200_FAIL(B200_ERR_MISSING, "decoder LM finalize: tensor '%s' [buckets, heads] was not loaded", name.c_str());
+  const int B = (int)t->shape[0], half = B / 2, H = a.heads;
+  if (!(a.bias_max > half)) B200_FAIL(B200_ERR_SHAPE, "decoder LM: layer %d: bias_max must be above half the bias table's rows", i);
+  auto bucket = [&](int n) {      // a quotient that is a whole number in exact arithmetic must not fall below it
+    if (n < half) return n;
+    return std::min(B - 1, half + (int)std::floor(std::log((double)n / half) / std::log((double)a.bias_max / half) * (B - half) + 1e-9));
+  };
+  L.far = 0;
+  while (bucket(L.far) < B - 1) ++L.far;
+  float* rel = nullptr;
+  B200_CUDA(cudaMalloc(&rel, (size_t)B * H * sizeof(float)));
+  int rc = convert_into(t, rel);
+  std::vector<float> src((size_t)B * H), dst((size_t)H * (L.far + 1));
+  if (rc == B200_OK && cudaMemcpy(src.data(), rel, src.size() * sizeof(float), cudaMemcpyDeviceToHost) != cudaSuccess) rc = B200_ERR_CUDA;
+  cudaFree(rel);
+  B200_TRY(rc);
+  for (int n = 0; n <= L.far; ++n) {
+    const int b = bucket(n);
+    for (int q = 0; q < H; ++q) dst[(size_t)q * (L.far + 1) + n] = src[(size_t)b * H + q];
+  }
+  B200_TRY(h->weights.alloc_t(&L.rel, dst.size(), false));
+  B200_CUDA(cudaMemcpy(L.rel, dst.data(), dst.size() * sizeof(float), cudaMemcpyHostToDevice));
+  h->weight_bytes += (int64_t)dst.size() * 4;
+  return B200_OK;
+}
+
+// Joint layers of the parallel-residual block (norm loaded already): every projection of the normed input is one matrix, both output
+// products are one; latent attention with a query latent, bias attention or RG-LRU, beside a silu-gated unit or gelu experts with a
+// shared one.
+int finalize_joint_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
+  Layer& L = h->layers[i];
+  const b200_dlm_config& c = h->cfg;
+  const b200_dlm_mixer& a = L.c.a;
+  const int64_t W = c.width;
+  const size_t es = esize(h);
+  const std::string p = "l" + std::to_string(i) + ".", m = p + "mix.";
+  auto pad8 = [](int v) { return (v + 7) / 8 * 8; };
+  auto matrix = [&](const std::string& name, int64_t rows, int64_t K, void** out) -> int {
+    B200_TRY(h->weights.alloc(out, (size_t)rows * K * es, false));
+    h->weight_bytes += rows * K * es;
+    return put_matrix(h, name, rows, K, *out);
+  };
+  const bool latent = L.c.mixer == B200_MIXER_LATENT_ATTENTION, bias_attn = L.c.mixer == B200_MIXER_BIAS_ATTENTION;
+  const bool dense = L.c.mlp == B200_MLP_DENSE_SILU_GLU, moe = L.c.mlp == B200_MLP_MOE_GELU;
+  const int H = a.heads, G = a.kv_heads, Kv = H * a.vdim;
+  L.glu_ff = dense ? L.c.ff : moe ? L.c.shared_ff : 0;
+  const std::string unit = p + (dense ? "mlp." : "mlp.shared.");
+  struct Part { std::string name; int rows; int* off; };
+  std::vector<Part> parts;
+  if (latent) {
+    L.Nq = H * (a.dim + a.rot_dims);
+    if (a.q_rank > 0) parts.push_back({m + "dq", a.q_rank, &L.off_q});
+    else parts.push_back({m + "q", L.Nq, &L.off_q});
+    parts.push_back({m + "dkv", a.kv_rank + a.rot_dims, &L.off_dkv});
+  } else if (bias_attn) {
+    L.Nq = H * a.dim; L.Nk = G * a.dim; L.Nv = G * a.vdim;
+    parts.push_back({m + "q", L.Nq, &L.p_q});
+    parts.push_back({m + "k", L.Nk, &L.p_k});
+    parts.push_back({m + "v", L.Nv, &L.p_v});
+  } else {
+    parts.push_back({m + "y", a.dim, &L.g_g});
+    parts.push_back({m + "x", a.dim, &L.g_x});
+  }
+  if (a.out_gate) parts.push_back({m + "g", Kv, &L.p_g});
+  if (dense) parts.push_back({unit + "gate", L.glu_ff, &L.p_ffg});
+  if (L.glu_ff) parts.push_back({unit + "up", L.glu_ff, &L.p_ffu});
+  L.ncat = 0;
+  for (auto& q : parts) { *q.off = pad8(L.ncat); L.ncat = *q.off + q.rows; }
+  if (!dense) L.p_ffg = L.p_ffu;
+  L.ldp = pad8(L.ncat);
+  void* cat = nullptr;
+  B200_TRY(h->weights.alloc(&cat, (size_t)L.ncat * W * es, true));
+  for (auto& q : parts) B200_TRY(put_matrix(h, q.name, q.rows, W, static_cast<char*>(cat) + (size_t)*q.off * W * es));
+  B200_TRY(seal_weight(h, L.cat, cat, L.ncat, (int)W, drop));
+  if (latent) {
+    const int r = a.kv_rank, rd = a.rot_dims;
+    L.rp = pad8(r + rd);
+    {   // bf16: rows padded to a multiple of 64 take the tensor-core kernel, when that costs at most a third more cache
+      const int rp64 = (r + rd + 63) / 64 * 64;
+      if (!h->f32 && h->use_tc && rp64 <= 576 && (int64_t)rp64 * 3 <= (int64_t)(r + rd) * 4) L.rp = rp64;
     }
-  if (!L.QT) B200_FAIL(B200_ERR_SHAPE, "decoder LM: layer %d: the attention's heads do not fit shared memory", i);
-  L.sig = add_sig(h, rep, L.QT);
-  if (!h->f32 && a.dim % 16 == 0 && a.vdim % 16 == 0 && a.vdim <= 128) {
-    L.mma_vt = ceil_div(a.vdim, 32) * 2;
-    L.mma_smem = diff_attn_mma_smem(a.dim, L.mma_vt, false);
-    L.smem_mma_one = diff_attn_mma_smem(a.dim, L.mma_vt, true);
-    if (std::max(L.mma_smem, L.smem_mma_one) <= 220 * 1024) { L.sig_mma = add_sig(h, rep, 64); L.sig_one = add_sig(h, rep, 16); }
+    if (a.q_rank > 0) {
+      B200_TRY(get_f32(h, m + "dq.norm", a.q_rank, &L.qnorm));
+      void *uq = nullptr, *tmp = nullptr;
+      const int ldk = pad8(a.q_rank);      // rows of the query latent start on 16 bytes
+      B200_TRY(h->weights.alloc(&uq, (size_t)L.Nq * ldk * es, true));
+      B200_CUDA(cudaMalloc(&tmp, (size_t)L.Nq * a.q_rank * es));
+      int rc = put_matrix(h, m + "uq", L.Nq, a.q_rank, tmp);
+      if (rc == B200_OK && cudaMemcpy2D(uq, (size_t)ldk * es, tmp, (size_t)a.q_rank * es, (size_t)a.q_rank * es, (size_t)L.Nq, cudaMemcpyDeviceToDevice) != cudaSuccess) rc = B200_ERR_CUDA;
+      cudaDeviceSynchronize();
+      cudaFree(tmp);
+      B200_TRY(rc);
+      B200_TRY(seal_weight(h, L.uq, uq, L.Nq, ldk, drop, pad8(L.Nq)));
+    }
+    B200_TRY(get_f32(h, m + "dkv.norm", r, &L.cnorm));
+    if (a.sink == B200_SINK_LEARNED) B200_TRY(get_f32(h, m + "sink", H, &L.sink));
+    else if (a.sink == B200_SINK_UNIT) B200_TRY(h->weights.alloc_t(&L.sink, (size_t)H, true));
+    {   // W_uk [H * dim][r] -> per head [r][dim]
+      void* uk = nullptr;
+      B200_TRY(matrix(m + "uk", (int64_t)H * a.dim, r, &uk));
+      B200_TRY(h->weights.alloc(&L.ukT, (size_t)H * a.dim * r * es, false));
+      const long long n = (long long)H * a.dim * r;
+      if (h->f32) B200_LAUNCH(head_transpose_kernel<float>, (unsigned)ceil_div64(n, 256), 256, 0, nullptr, static_cast<const float*>(uk), static_cast<float*>(L.ukT), H, a.dim, r);
+      else B200_LAUNCH(head_transpose_kernel<bf16>, (unsigned)ceil_div64(n, 256), 256, 0, nullptr, static_cast<const bf16*>(uk), static_cast<bf16*>(L.ukT), H, a.dim, r);
+      B200_TRY(check_launch("head_transpose"));
+      drop.push_back(uk);
+    }
+    B200_TRY(matrix(m + "uv", Kv, r, &L.uv));
+    B200_TRY(add_rotation(h, a, &L.rot_id));
+    L.sig = add_sig(h, H, rows_per_tile(L.rp));
+  } else if (bias_attn) {
+    if (a.bias) {
+      const int C = L.Nq + L.Nk + L.Nv;
+      B200_TRY(h->weights.alloc_t(&L.qkv_bias, (size_t)C, false));
+      const Tensor* t = nullptr;
+      int off = 0;
+      for (const char* nm : {"q", "k", "v"}) {
+        const int rows = nm[0] == 'q' ? L.Nq : nm[0] == 'k' ? L.Nk : L.Nv;
+        B200_TRY(find_tensor(h, m + nm + ".b", {rows}, &t));
+        B200_TRY(convert_into(t, L.qkv_bias + off));
+        off += rows;
+      }
+      h->weight_bytes += (int64_t)C * 4;
+    }
+    if (a.qk_norm) {
+      B200_TRY(get_f32(h, m + "q.norm", a.dim, &L.qnorm));
+      B200_TRY(get_f32(h, m + "k.norm", a.dim, &L.knorm));
+    }
+    B200_TRY(put_distance_bias(h, m + "rel", L, i));
+    B200_TRY(plan_map_attention(h, L, i, 1));
+  } else {
+    const int n = a.dim, nb = a.blocks, bs = n / nb;
+    B200_TRY(get_f32(h, m + "x.b", n, &L.x_b));
+    B200_TRY(get_f32(h, m + "y.b", n, &L.y_b));
+    B200_TRY(get_f32_shaped(h, m + "conv", {n, a.conv_taps}, &L.qkv_conv));
+    B200_TRY(get_f32(h, m + "conv.b", n, &L.conv_b));
+    float *lam = nullptr, *rb = nullptr, *ib = nullptr;
+    B200_TRY(get_f32(h, m + "lam", n, &lam));
+    B200_TRY(h->weights.alloc_t(&L.lam8, (size_t)n, false));
+    B200_LAUNCH(rglru_decay_kernel, ceil_div(n, 256), 256, 0, nullptr, lam, L.lam8, n);
+    B200_TRY(get_f32_shaped(h, m + "ra.b", {nb, bs}, &rb));
+    B200_TRY(get_f32_shaped(h, m + "ri.b", {nb, bs}, &ib));
+    B200_TRY(h->weights.alloc_t(&L.gate_b, (size_t)2 * n, false));
+    B200_LAUNCH(interleave_pairs_kernel, ceil_div(n, 256), 256, 0, nullptr, rb, ib, L.gate_b, n);
+    // rows 2c / 2c + 1 of a block are its matrices' rows c for r / i
+    const Tensor *ta = nullptr, *ti = nullptr;
+    B200_TRY(find_tensor(h, m + "ra", {nb, bs, bs}, &ta));
+    B200_TRY(find_tensor(h, m + "ri", {nb, bs, bs}, &ti));
+    void *ra = nullptr, *ri = nullptr;
+    B200_TRY(h->weights.alloc(&ra, (size_t)n * bs * es, false));
+    B200_TRY(h->weights.alloc(&ri, (size_t)n * bs * es, false));
+    B200_TRY(h->weights.alloc(&L.gates, (size_t)2 * n * bs * es, false));
+    const unsigned g = (unsigned)ceil_div64((int64_t)n * bs, 256);
+    if (h->f32) {
+      B200_TRY(convert_into(ta, static_cast<float*>(ra))); B200_TRY(convert_into(ti, static_cast<float*>(ri)));
+      B200_LAUNCH(interleave_rows_kernel<float>, g, 256, 0, nullptr, static_cast<const float*>(ra), static_cast<const float*>(ri), static_cast<float*>(L.gates), (long long)n, (long long)bs);
+    } else {
+      B200_TRY(convert_into(ta, static_cast<bf16*>(ra))); B200_TRY(convert_into(ti, static_cast<bf16*>(ri)));
+      B200_LAUNCH(interleave_rows_kernel<bf16>, g, 256, 0, nullptr, static_cast<const bf16*>(ra), static_cast<const bf16*>(ri), static_cast<bf16*>(L.gates), (long long)n, (long long)bs);
+    }
+    B200_TRY(check_launch("RG-LRU gate matrices"));
+    drop.push_back(ra); drop.push_back(ri);
+    h->weight_bytes += (int64_t)2 * n * bs * es;
+  }
+  if (moe) {
+    const int64_t E = L.c.experts, F = L.c.ff;
+    L.s_router = 0; L.nsmall = (int)E;
+    B200_TRY(matrix(p + "mlp.router", E, W, &L.w_small));
+    B200_TRY(get_f32(h, p + "mlp.correction", E, &L.correction));
+    B200_TRY(h->weights.alloc(&L.ups, (size_t)E * F * W * es, false));
+    B200_TRY(h->weights.alloc(&L.downs, (size_t)E * W * F * es, false));
+    for (int64_t e = 0; e < E; ++e) {
+      const std::string q = p + "mlp.e" + std::to_string(e) + ".";
+      B200_TRY(put_matrix(h, q + "up", F, W, static_cast<char*>(L.ups) + (size_t)e * F * W * es));
+      B200_TRY(put_matrix(h, q + "down", W, F, static_cast<char*>(L.downs) + (size_t)e * W * F * es));
+    }
+    h->weight_bytes += 2 * E * F * W * es;
+  }
+  B200_TRY(put_joint_output(h, L, m + "o", unit + "down", Kv, drop));
+  if (c.side_dim > 0) {
+    const int D = c.side_dim;
+    B200_TRY(matrix(p + "side.gate", D, W, &L.side_gate_rm));
+    L.side_gate.rm = L.side_gate_rm; L.side_gate.N = D; L.side_gate.K = (int)W;      // kept row-major as well: the few-token kernel reads it
+    if (!h->f32 && h->use_tc && W % 8 == 0 && (D + 127) / 128 <= tc::SK_MAX_TILES) {
+      B200_TRY(h->weights.alloc(&L.side_gate.tiles, tc::sk_packed_bytes(D, (int)W, 0, 0), false));
+      B200_TRY(tc::sk_pack_weights(static_cast<const bf16*>(L.side_gate_rm), L.side_gate.tiles, D, (int)W, 0, 0, nullptr));
+    }
+    void *proj = nullptr, *tmp = nullptr;
+    B200_TRY(h->weights.alloc(&proj, (size_t)W * h->side_ld * es, true));
+    B200_CUDA(cudaMalloc(&tmp, (size_t)W * D * es));
+    int rc = put_matrix(h, p + "side.proj", W, D, tmp);
+    if (rc == B200_OK && cudaMemcpy2D(proj, (size_t)h->side_ld * es, tmp, (size_t)D * es, (size_t)D * es, (size_t)W, cudaMemcpyDeviceToDevice) != cudaSuccess) rc = B200_ERR_CUDA;
+    cudaDeviceSynchronize();
+    cudaFree(tmp);
+    B200_TRY(rc);
+    B200_TRY(seal_weight(h, L.side_proj, proj, (int)W, h->side_ld, drop, (int)W));
+    B200_TRY(get_f32(h, p + "side.norm", W, &L.side_norm));
   }
   return B200_OK;
 }
@@ -1159,6 +1411,7 @@ int finalize_parallel_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
   B200_TRY(get_f32(h, p + "norm1", W, &L.n1w));
   if (c.norm == B200_NORM_RMS_ZERO_CENTRED) B200_LAUNCH(add_one_kernel, ceil_div((int)W, 256), 256, 0, nullptr, L.n1w, (int)W);
   if (L.c.mixer == B200_MIXER_DIFF_ATTENTION) return finalize_diff_layer(h, i, drop);
+  if (L.c.mixer == B200_MIXER_LATENT_ATTENTION || L.c.mixer == B200_MIXER_BIAS_ATTENTION || L.c.mixer == B200_MIXER_RGLRU) return finalize_joint_layer(h, i, drop);
   const bool attn = L.c.mixer == B200_MIXER_SIGMOID_ATTENTION, ret = L.c.mixer == B200_MIXER_RETENTION, delta = L.c.mixer == B200_MIXER_DELTA;
   const int H = a.heads, G = attn || delta ? a.kv_heads : a.heads;
   L.Nq = (attn ? H : G) * a.dim; L.Nk = G * a.dim; L.Nv = (attn ? G : H) * a.vdim;
@@ -1324,104 +1577,219 @@ int sigmoid_attention(b200_dlm* h, const Layer& L, int n_tok, int max_ctx) {
   return B200_OK;
 }
 
-template <int VT, bool SK>
-int launch_diff_mma(cudaStream_t st, const DiffAttnParams& p, size_t smem) {
+constexpr int SIDE_FEW = 64;      // up to this many tokens the token input's gate product runs from the fp32 residual in one launch
+
+// the gated unit of a layer whose preparation carries it: columns of the projection -> second half of the output product's rows
+template <typename T>
+UnitParams unit_params(b200_dlm* h, const Layer& L) {
+  UnitParams u;
+  u.off_g = L.p_ffg; u.off_u = L.p_ffu; u.F = L.glu_ff; u.limit = L.c.expert_limit;
+  u.kind = L.c.mlp == B200_MLP_DENSE_CLAMPED_GLU ? GLU_CLAMPED : L.c.mlp == B200_MLP_MOE_GELU ? UNIT_GELU_ERF : GLU_SILU;
+  u.act = static_cast<T*>(h->obuf) + L.ob_act; u.lda = L.ob_ld;
+  return u;
+}
+
+template <int NM, int VT, bool SK>
+int launch_map_mma(cudaStream_t st, const MapAttnParams& p, size_t smem) {
   static bool attr_set = false;
   if (!attr_set) {
-    B200_CUDA(cudaFuncSetAttribute((diff_attn_mma_kernel<VT, SK>), cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    B200_CUDA(cudaFuncSetAttribute((map_attn_mma_kernel<NM, VT, SK>), cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     attr_set = true;
   }
-  B200_LAUNCH((diff_attn_mma_kernel<VT, SK>), dim3(p.n_tiles * p.G, p.nsplit), 128, smem, st, p);
-  return check_launch("diff_attn_mma");
+  B200_LAUNCH((map_attn_mma_kernel<NM, VT, SK>), dim3(p.n_tiles * p.G, p.nsplit), 128, smem, st, p);
+  return check_launch("map_attn_mma");
 }
 
-template <bool SK>
-int launch_diff_mma_vt(cudaStream_t st, const DiffAttnParams& p, int vt, size_t smem) {
+template <int NM, bool SK>
+int launch_map_mma_vt(cudaStream_t st, const MapAttnParams& p, int vt, size_t smem) {
   switch (vt) {
-    case 2: return launch_diff_mma<2, SK>(st, p, smem);
-    case 4: return launch_diff_mma<4, SK>(st, p, smem);
-    case 6: return launch_diff_mma<6, SK>(st, p, smem);
-    default: return launch_diff_mma<8, SK>(st, p, smem);
+    case 2: return launch_map_mma<NM, 2, SK>(st, p, smem);
+    case 4: return launch_map_mma<NM, 4, SK>(st, p, smem);
+    case 6: return launch_map_mma<NM, 6, SK>(st, p, smem);
+    case 8: return launch_map_mma<NM, 8, SK>(st, p, smem);
   }
+  if constexpr (NM == 1) {
+    if (vt <= 12) return launch_map_mma<1, 12, SK>(st, p, smem);
+    return launch_map_mma<1, 16, SK>(st, p, smem);
+  }
+  B200_FAIL(B200_ERR_SHAPE, "decoder LM: no attention kernel for %d value columns", vt * 16);
 }
 
-// which attention kernel a step takes: the tensor cores (16-row tiles whose warps share the keys when no request brings more rows), or the CUDA cores
-template <typename T>
-bool diff_attention_on_tensor_cores(const b200_dlm* h, const Layer& L) { return sizeof(T) == 2 && h->attn_tc && L.sig_mma >= 0; }
-
-// gate and up of the gated unit, queries, keys and values from the projection; then the attention -> obuf [tokens][ob_ld]
-template <typename T>
-int diff_attention(b200_dlm* h, const Layer& L, int n_tok, int max_ctx) {
+// gate and up of the gated unit, queries, keys and values from the projection; then the attention with NM maps -> obuf [tokens][ob_ld]
+template <typename T, int NM>
+int map_attention(b200_dlm* h, const Layer& L, int n_tok, int max_ctx) {
   const b200_dlm_mixer& a = L.c.a;
-  const Layer& S = h->layers[L.kv_src];
+  const Layer& S = L.kv_src >= 0 ? h->layers[L.kv_src] : L;
   cudaStream_t st = h->stream;
-  const bool mma = diff_attention_on_tensor_cores<T>(h, L), own = a.kv_from < 0;
+  const bool mma = sizeof(T) == 2 && h->attn_tc && L.sig_mma >= 0, own = a.kv_from < 0;      // the tensor cores (16-row tiles whose warps share the keys when no request brings more rows), or the CUDA cores
   const int rep = a.heads / a.kv_heads;
   {
-    DiffPrepParams p;
-    p.proj = h->proj; p.ld = L.ldp; p.off_q = L.p_q; p.off_k = own ? L.p_k : -1; p.off_v = L.p_v; p.Hm = 2 * a.heads; p.Gm = 2 * a.kv_heads; p.Nv = L.Nv;
+    HeadPrepParams p;
+    p.proj = h->proj; p.ld = L.ldp; p.off_q = L.p_q; p.off_k = own ? L.p_k : -1; p.off_v = L.p_v; p.Hm = NM * a.heads; p.Gm = NM * a.kv_heads; p.Nv = L.Nv;
     p.dim = a.dim; p.half = a.rot_dims / 2; p.adjacent = a.rot_pairing == B200_ROT_ADJACENT; p.rot = L.rot_id >= 0 ? h->rots[L.rot_id].table : nullptr;
     p.bias = L.qkv_bias; p.wq = L.qnorm; p.wk = L.knorm; p.eps = h->cfg.norm_eps; p.qscale = a.scale; p.qout = h->qkv32;
     p.kcache = S.kcache; p.vcache = S.vcache; p.cap = h->cap; p.tok_slot = h->meta_dev + h->off_slot; p.tok_pos = h->meta_dev + h->off_pos;
-    p.off_g = L.p_ffg; p.off_u = L.p_ffu; p.F = L.glu_ff; p.glu = L.c.mlp == B200_MLP_DENSE_CLAMPED_GLU ? GLU_CLAMPED : GLU_SILU; p.limit = L.c.expert_limit;
-    p.act = static_cast<T*>(h->obuf) + L.ob_act; p.lda = L.ob_ld;
+    p.unit = unit_params<T>(h, L);
+    p.temp_coef = a.q_temp_coef; p.temp_every = a.q_temp_every;
     p.head_rows = n_tok >= 512 ? 1 : ceil_div(p.Hm + (own ? p.Gm : 0), 8);      // few tokens: one (head, map) per warp
     const dim3 grid(n_tok, p.head_rows + ceil_div(L.glu_ff, GLU_SLICE));
     const size_t smem = (size_t)8 * a.dim * sizeof(float);
-    TIMED(CLS_ELEMENTWISE, if (mma) B200_LAUNCH((diff_prep_kernel<T, bf16>), grid, 256, smem, st, p); else B200_LAUNCH((diff_prep_kernel<T, float>), grid, 256, smem, st, p));
-    B200_TRY(check_launch("diff_prep"));
+    TIMED(CLS_ELEMENTWISE, if (mma) B200_LAUNCH((head_prep_kernel<T, bf16>), grid, 256, smem, st, p); else B200_LAUNCH((head_prep_kernel<T, float>), grid, 256, smem, st, p));
+    B200_TRY(check_launch("head_prep"));
   }
   const bool one = mma && h->max_entry_tokens * rep <= 16;
   const TileSig& s = h->sigs[one ? L.sig_one : mma ? L.sig_mma : L.sig];
-  DiffAttnParams p;
+  MapAttnParams p;
   p.q = h->qkv32; p.ldq = L.Nq; p.kcache = S.kcache; p.vcache = S.vcache;
   p.tile_row0 = h->meta_dev + s.off_row0; p.tile_rows = h->meta_dev + s.off_rows; p.tile_slot = h->meta_dev + s.off_slot; p.tok_pos = h->meta_dev + h->off_pos;
   p.gate = a.head_gate ? h->small32 + L.s_gate : nullptr; p.ldg = L.nsmall; p.out = h->obuf; p.ldo = L.ob_ld; p.part = h->part;
   p.cap = h->cap; p.H = a.heads; p.G = a.kv_heads; p.dim = a.dim; p.vdim = a.vdim; p.chunk = a.chunk; p.n_tiles = s.count; p.MR = s.rpt; p.KT = mma ? DA_KT : L.KT;
   p.lambda = L.lambda; p.out_scale = 1.f - a.diff; p.eps = h->cfg.norm_eps;
+  p.bias = L.rel; p.far = L.far;
+  if (a.out_gate) { p.egate = static_cast<const T*>(h->proj) + L.p_g; p.lde = L.ldp; }
+  if (mma && L.far_smem) p.bias_smem = (int)((one ? L.smem_mma_one : L.mma_smem) - (size_t)rep * (L.far + 1) * 4);
   // keys are cut over several CTAs per tile when the tiles alone cannot fill the GPU (decoding, short portions)
   const int seen = a.chunk > 0 ? std::min(max_ctx, a.chunk + s.rpt / rep) : max_ctx, key_tiles = ceil_div(seen, p.KT), ctas = s.count * a.kv_heads;
   int nsplit = 1;
   if (h->attn_split > 0) nsplit = std::min(h->attn_split, 64);
   else if (ctas < 296) nsplit = std::min(296 / ctas, 64);
   nsplit = a.vdim > 1024 ? 1 : std::max(1, std::min(nsplit, key_tiles));
-  while (nsplit > 1 && (size_t)ctas * nsplit * s.rpt * (2 * a.vdim + 4) > h->part_floats) --nsplit;
+  while (nsplit > 1 && (size_t)ctas * nsplit * s.rpt * NM * (a.vdim + 2) > h->part_floats) --nsplit;
   p.nsplit = nsplit;
   B200_TRY(mark(h, CLS_ATTN));
   if (mma) {
-    if constexpr (sizeof(T) == 2) B200_TRY(one ? launch_diff_mma_vt<true>(st, p, L.mma_vt, L.smem_mma_one) : launch_diff_mma_vt<false>(st, p, L.mma_vt, L.mma_smem));
+    if constexpr (sizeof(T) == 2) B200_TRY(one ? (launch_map_mma_vt<NM, true>(st, p, L.mma_vt, L.smem_mma_one)) : (launch_map_mma_vt<NM, false>(st, p, L.mma_vt, L.mma_smem)));
   } else {
     static bool attr_set = false;
     if (!attr_set) {
-      B200_CUDA(cudaFuncSetAttribute(diff_attn_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+      B200_CUDA(cudaFuncSetAttribute((map_attn_kernel<T, NM>), cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
       attr_set = true;
     }
-    B200_LAUNCH(diff_attn_kernel<T>, dim3(ctas, nsplit), 256, L.attn_smem, st, p);
-    B200_TRY(check_launch("diff_attn"));
+    B200_LAUNCH((map_attn_kernel<T, NM>), dim3(ctas, nsplit), 256, L.attn_smem, st, p);
+    B200_TRY(check_launch("map_attn"));
   }
   if (nsplit > 1) {
-    B200_LAUNCH(diff_attn_merge_kernel<T>, dim3(ctas, ceil_div(s.rpt, 4)), 128, 0, st, p);
-    B200_TRY(check_launch("diff_attn_merge"));
+    B200_LAUNCH((map_attn_merge_kernel<T, NM>), dim3(ctas, ceil_div(s.rpt, 4)), 128, 0, st, p);
+    B200_TRY(check_launch("map_attn_merge"));
   }
   return mark(h, -1);
 }
 
-// routed gated experts on the rows of hb -> yexp [tokens * top][W]; the router's logits are in small32
+// latent attention with a query latent -> obuf [tokens][ob_ld]; the feed-forward's unit rides in the preparation
+template <typename T>
+int joint_latent_attention(b200_dlm* h, const Layer& L, int n_tok, int max_ctx) {
+  const b200_dlm_mixer& a = L.c.a;
+  const int H = a.heads, dk = a.dim, dv = a.vdim, r = a.kv_rank, rd = a.rot_dims, rp = L.rp;
+  cudaStream_t st = h->stream;
+  const int* meta = h->meta_dev;
+  T* proj = static_cast<T*>(h->proj);
+  const float* rot = L.rot_id >= 0 ? h->rots[L.rot_id].table : nullptr;
+  LatentPrepParams lp;
+  lp.proj = proj; lp.ld = L.ldp; lp.off_dq = L.off_q; lp.q_rank = a.q_rank; lp.off_dkv = L.off_dkv; lp.r = r; lp.rd = rd; lp.rp = rp;
+  lp.adjacent = a.rot_pairing == B200_ROT_ADJACENT; lp.wq = L.qnorm; lp.wc = L.cnorm; lp.cq = h->cq; lp.ldc = (a.q_rank + 7) / 8 * 8;
+  lp.cache = L.cache; lp.cap = h->cap; lp.rot = rot; lp.tok_slot = meta + h->off_slot; lp.tok_pos = meta + h->off_pos; lp.eps = h->cfg.norm_eps;
+  lp.unit = unit_params<T>(h, L);
+  TIMED(CLS_ELEMENTWISE, B200_LAUNCH(latent_prep_kernel<T>, dim3(n_tok, 1 + ceil_div(L.glu_ff, GLU_SLICE)), 256, 0, st, lp));
+  const T* q = proj + L.off_q;
+  long long ldq = L.ldp;
+  if (a.q_rank > 0) {
+    ldq = (L.Nq + 7) / 8 * 8;
+    TIMED(CLS_LINEAR, B200_TRY(linear<T>(h, static_cast<const T*>(h->cq), lp.ldc, L.uq, static_cast<T*>(h->q2), ldq, n_tok)));
+    q = static_cast<const T*>(h->q2);
+  }
+  if (rp > r) TIMED(CLS_ELEMENTWISE, B200_LAUNCH(latent_query_rope_kernel<T>, n_tok, 128, 0, st, q, ldq, H, dk, rd, r, rp, lp.adjacent, rot, a.scale, h->qa));
+  TIMED(CLS_FOLD, B200_TRY(head_gemm(st, q, ldq, (long long)(dk + rd), static_cast<const T*>(L.ukT), (long long)dk, (long long)r * dk, h->qa,
+                                     (long long)H * rp, (long long)rp, n_tok, r, dk, H, a.scale, h->attn_tc != 0)));
+  const TileSig& s = h->sigs[L.sig];
+  AttnParams p;
+  p.qa = h->qa; p.cache = L.cache; p.sink = a.sink == B200_SINK_NONE ? nullptr : L.sink;
+  p.tile_row0 = meta + s.off_row0; p.tile_rows = meta + s.off_rows; p.tile_slot = meta + s.off_slot; p.tok_pos = meta + h->off_pos;
+  p.out = h->ol; p.part = h->part; p.cap = h->cap; p.r = rp; p.H = H; p.err = h->err;
+  p.window = a.window;
+  p.nsplit = pick_split(h->attn_split, s.count, a.window > 0 ? std::min(max_ctx, a.window + 32) : max_ctx, s.rpt, rp, h->part_floats);
+  TIMED(CLS_ATTN, B200_TRY(run_attention<T>(st, p, s.count, s.rpt, h->attn_tc != 0)));
+  TIMED(CLS_FOLD, B200_TRY(head_gemm(st, h->ol, (long long)H * rp, (long long)rp, static_cast<const T*>(L.uv), (long long)r, (long long)dv * r, static_cast<T*>(h->obuf),
+                                     (long long)L.ob_ld, (long long)dv, n_tok, dv, r, H, 1.f, h->attn_tc != 0, a.out_gate ? proj + L.p_g : (const T*)nullptr, (long long)L.ldp, (long long)dv)));
+  return B200_OK;
+}
+
+// RG-LRU -> obuf [tokens][ob_ld]; the feed-forward's unit rides in the convolution
+template <typename T>
+int rglru(b200_dlm* h, const Layer& L, int n_tok) {
+  const b200_dlm_mixer& a = L.c.a;
+  cudaStream_t st = h->stream;
+  const int* meta = h->meta_dev;
+  RgLruParams p;
+  p.proj = h->proj; p.ld = L.ldp; p.off_x = L.g_x; p.off_y = L.g_g; p.C = a.dim; p.taps = a.conv_taps; p.bs = a.dim / a.blocks;
+  p.bx = L.x_b; p.by = L.y_b; p.conv = L.qkv_conv; p.bc = L.conv_b; p.hist = L.qkv_hist; p.u = h->qkv32; p.gates = L.gates; p.gate_b = L.gate_b; p.lam8 = L.lam8;
+  p.ab = reinterpret_cast<float2*>(h->gate32); p.state = L.gru; p.out = h->obuf; p.ldo = L.ob_ld;
+  p.tok_slot = meta + h->off_slot; p.tok_pos = meta + h->off_pos; p.tok_first = meta + h->off_first; p.tok_last = meta + h->off_last;
+  p.ent_tok0 = meta + h->off_whole_tok0; p.ent_ntok = meta + h->off_whole_ntok; p.ent_slot = meta + h->off_whole_slot; p.ent_pos0 = meta + h->off_whole_pos0;
+  p.n_tok = n_tok; p.unit = unit_params<T>(h, L); p.conv_rows = ceil_div(p.C, CONV_SLICE);
+  TIMED(CLS_ELEMENTWISE, B200_LAUNCH(rglru_conv_kernel<T>, dim3(n_tok, p.conv_rows + ceil_div(L.glu_ff, GLU_SLICE)), 256, 0, st, p);
+        if (p.taps > 1 && h->max_entry_tokens > 1)
+          B200_LAUNCH(conv_carry_kernel<T>, n_tok, 256, 0, st, static_cast<const T*>(h->proj) + L.g_x, (long long)L.ldp, L.qkv_hist, p.C, p.taps - 1, p.tok_slot, p.tok_pos,
+                      p.tok_last, L.x_b));
+  B200_TRY(check_launch("rglru_conv"));
+  const bool mma = sizeof(T) == 2 && h->attn_tc && p.bs % 16 == 0, single = mma && h->max_entry_tokens == 1;
+  if (mma) {
+    const dim3 grid(ceil_div(2 * p.bs, 64), ceil_div(n_tok, 64), a.blocks);
+    if (single) TIMED(CLS_RECURRENT, B200_LAUNCH(rglru_gates_mma_kernel<true>, grid, 128, 0, st, p));
+    else TIMED(CLS_RECURRENT, B200_LAUNCH(rglru_gates_mma_kernel<false>, grid, 128, 0, st, p));
+  } else {
+    TIMED(CLS_RECURRENT, B200_TRY(gemm_nt(st, static_cast<const float*>(p.u), (long long)p.C, (long long)p.bs, static_cast<const T*>(p.gates), (long long)p.bs, (long long)2 * p.bs * p.bs,
+                                          h->gate32, (long long)2 * p.C, (long long)2 * p.bs, n_tok, 2 * p.bs, p.bs, a.blocks, 1.f));
+          B200_LAUNCH(rglru_coefficients_kernel, (unsigned)ceil_div64((int64_t)n_tok * p.C, 256), 256, 0, st, p));
+  }
+  B200_TRY(check_launch("rglru_gates"));
+  if (single) return B200_OK;
+  // segments of at least 8 tokens, as many as fill 1024 threads: 16 channels x 64 segments for a prompt, 128 channels x 1 for single tokens
+  int ns = 1;
+  while (ns < 64 && ns * 16 <= h->max_entry_tokens) ns *= 2;
+  const int nx = std::max(16, 128 / ns);
+  TIMED(CLS_RECURRENT, B200_LAUNCH(rglru_scan_kernel<T>, dim3(ceil_div(p.C, nx), h->n_entries), dim3(nx, ns), (size_t)2 * nx * ns * sizeof(float), st, p));
+  return check_launch("rglru_scan");
+}
+
+// the per-layer token input and the end of the block behind it: x += rms(W_proj (gelu(W_gate x) * e)) * w, trace, step vector, next norm
+template <typename T>
+int token_input(b200_dlm* h, const Layer& L, int n_tok, float* trace, const float* step, const float* w_next) {
+  const int W = h->cfg.width, D = h->cfg.side_dim, off = L.index * D;
+  cudaStream_t st = h->stream;
+  const int* tok = h->meta_dev + h->off_tok;
+  T *z = static_cast<T*>(h->sidez), *hb = static_cast<T*>(h->hbuf), *y = static_cast<T*>(h->mixo);
+  const T* table = static_cast<const T*>(h->side_embed);
+  if (n_tok <= SIDE_FEW) {
+    TIMED(CLS_FOLD, B200_LAUNCH(side_gate_kernel<T>, dim3(n_tok, ceil_div(D, 8)), 256, 0, st, h->xin, W, static_cast<const T*>(L.side_gate_rm), table, (long long)h->side_cols, off, tok,
+                                h->cfg.vocab, D, z, (long long)h->side_ld, W % 8 == 0));
+  } else {
+    TIMED(CLS_FOLD, B200_TRY(linear<T>(h, hb, W, L.side_gate, z, h->side_ld, n_tok));
+          B200_LAUNCH(side_act_kernel<T>, (unsigned)ceil_div64((int64_t)n_tok * D, 256), 256, 0, st, z, (long long)h->side_ld, table, (long long)h->side_cols, off, tok, h->cfg.vocab, D,
+                      (long long)n_tok * D));
+  }
+  TIMED(CLS_FOLD, B200_TRY(linear<T>(h, z, (long long)h->side_ld, L.side_proj, y, W, n_tok)));
+  auto end = n_tok <= 592 && W <= 4096 ? side_end_kernel<T, true> : side_end_kernel<T, false>;
+  TIMED(CLS_ELEMENTWISE, B200_LAUNCH(end, n_tok, 256, 0, st, h->xin, y, L.side_norm, trace, step, w_next, hb, W, h->cfg.norm_eps));
+  return check_launch("token_input");
+}
+
+// routed experts (gated, or with an erf GELU) on the rows of hb -> yexp [tokens * top][W]; the router's logits are in small32
 template <typename T>
 int routed_experts_glu(b200_dlm* h, const Layer& L, const T* hb, int n_tok) {
   const int W = h->cfg.width, E = L.c.experts, top = L.c.top, F = L.c.ff, pairs = n_tok * top;
-  const bool silu = L.c.mlp == B200_MLP_MOE_SILU_GLU;
+  const bool silu = L.c.mlp == B200_MLP_MOE_SILU_GLU, gelu = L.c.mlp == B200_MLP_MOE_GELU;
+  const int N1 = gelu ? F : 2 * F;       // rows of an expert's first matrix
   cudaStream_t st = h->stream;
-  if (silu) {
+  if (silu || gelu) {
     const int n = E + L.c.identity, groups = std::max(L.c.groups, 1);
     const size_t smem = (size_t)4 * (2 * n + groups) * sizeof(float);
     static bool attr_set = false;
     if (!attr_set) {
-      B200_CUDA(cudaFuncSetAttribute(moe_route_softmax_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+      B200_CUDA(cudaFuncSetAttribute(moe_route_grouped_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
       attr_set = true;
     }
-    B200_LAUNCH(moe_route_softmax_kernel, ceil_div(n_tok, 4), 128, smem, st, h->small32 + L.s_router, (long long)L.nsmall, L.correction, n, top, groups, L.c.groups_keep,
-                h->moe_idx, h->moe_w, n_tok);
+    B200_LAUNCH(moe_route_grouped_kernel, ceil_div(n_tok, 4), 128, smem, st, h->small32 + L.s_router, (long long)L.nsmall, L.correction, n, top, groups, L.c.groups_keep,
+                gelu ? 1 : 0, gelu ? 2 : 1, gelu ? 1 : 0, L.c.router_scale, h->moe_idx, h->moe_w, n_tok);
   } else {
     B200_LAUNCH(moe_route_sigmoid_kernel, ceil_div(n_tok, 4), 128, 0, st, h->small32 + L.s_router, (long long)L.nsmall, L.correction, E, top, L.c.router_scale,
                 h->moe_idx, h->moe_w, n_tok);
@@ -1447,15 +1815,15 @@ int routed_experts_glu(b200_dlm* h, const Layer& L, const T* hb, int n_tok) {
         attr_set = true;
       }
       // gate and value rows of an expert are interleaved, so the first product's epilogue holds both of an output in one thread
-      B200_LAUNCH(grouped_gemm_mma_kernel, dim3(ceil_div(2 * F, 128), max_tiles), 256, GG_SMEM, st, hb, (long long)W, h->moe_row_tok, ups, (long long)W, (long long)2 * F * W,
-                  act, (long long)F, (const int*)nullptr, h->moe_tile_e, h->moe_tile_r0, h->moe_tile_n, h->moe_ntiles, 2 * F, W, silu ? 3 : 2, L.c.expert_limit);
+      B200_LAUNCH(grouped_gemm_mma_kernel, dim3(ceil_div(N1, 128), max_tiles), 256, GG_SMEM, st, hb, (long long)W, h->moe_row_tok, ups, (long long)W, (long long)N1 * W,
+                  act, (long long)F, (const int*)nullptr, h->moe_tile_e, h->moe_tile_r0, h->moe_tile_n, h->moe_ntiles, N1, W, gelu ? 4 : silu ? 3 : 2, L.c.expert_limit);
       B200_LAUNCH(grouped_gemm_mma_kernel, dim3(ceil_div(W, 128), max_tiles), 256, GG_SMEM, st, act, (long long)F, (const int*)nullptr, downs, (long long)F, (long long)W * F,
                   yexp, (long long)W, h->moe_perm, h->moe_tile_e, h->moe_tile_r0, h->moe_tile_n, h->moe_ntiles, W, F, 0, 0.f);
     }
   } else {
-    B200_LAUNCH((grouped_gemm_kernel<T, T, T>), dim3(ceil_div(2 * F, 64), max_tiles), 256, 0, st, hb, (long long)W, h->moe_row_tok, ups, (long long)W, (long long)2 * F * W,
-                act2, (long long)2 * F, (const int*)nullptr, h->moe_tile_e, h->moe_tile_r0, h->moe_tile_n, h->moe_ntiles, 2 * F, W, 0);
-    B200_LAUNCH(interleaved_glu_kernel<T>, (unsigned)ceil_div64(n, 256), 256, 0, st, act2, act, F, n, L.c.expert_limit, silu ? 1 : 0);
+    B200_LAUNCH((grouped_gemm_kernel<T, T, T>), dim3(ceil_div(N1, 64), max_tiles), 256, 0, st, hb, (long long)W, h->moe_row_tok, ups, (long long)W, (long long)N1 * W,
+                gelu ? act : act2, (long long)N1, (const int*)nullptr, h->moe_tile_e, h->moe_tile_r0, h->moe_tile_n, h->moe_ntiles, N1, W, gelu ? 4 : 0);
+    if (!gelu) B200_LAUNCH(interleaved_glu_kernel<T>, (unsigned)ceil_div64(n, 256), 256, 0, st, act2, act, F, n, L.c.expert_limit, silu ? 1 : 0);
     B200_LAUNCH((grouped_gemm_kernel<T, T, T>), dim3(ceil_div(W, 64), max_tiles), 256, 0, st, act, (long long)F, (const int*)nullptr, downs, (long long)F, (long long)W * F,
                 yexp, (long long)W, h->moe_perm, h->moe_tile_e, h->moe_tile_r0, h->moe_tile_n, h->moe_ntiles, W, F, 0);
   }
@@ -1535,19 +1903,26 @@ int step_parallel(b200_dlm* h, int n_tok, int n_want, int max_ctx, float* logits
   T* ob = static_cast<T*>(h->obuf);
   T* mixo = static_cast<T*>(h->mixo);
   TIMED(CLS_ELEMENTWISE, B200_LAUNCH(embed_scale_norm_kernel<T>, n_tok, 256, 0, st, meta + h->off_tok, static_cast<const T*>(h->embed), c.vocab, W, c.embedding_scale,
-                                     h->layers[0].n1w, h->xin, hb, c.norm_eps, h->err, c.norm == B200_NORM_LAYER));
+                                     h->layers[0].n1w, h->xin, hb, c.norm_eps, h->err, c.norm == B200_NORM_LAYER, h->layers[0].step));
   for (const auto& r : h->rots)
-    TIMED(CLS_ELEMENTWISE, B200_LAUNCH(rotary_table_kernel, n_tok, 64, 0, st, tok_pos, r.freq, r.m.rot_dims / 2, 1.f, r.table));
-  for (int li = 0; li < c.n_layers; ++li) {
+    TIMED(CLS_ELEMENTWISE, B200_LAUNCH(rotary_table_kernel, n_tok, 64, 0, st, tok_pos, r.freq, r.m.rot_dims / 2, r.amp, r.table));
+  const int n_runs = (int)h->layers.size();
+  for (int li = 0; li < n_runs; ++li) {
     const Layer& L = h->layers[li];
     const b200_dlm_mixer& a = L.c.a;
-    const bool last = li + 1 == c.n_layers;
+    const bool last = li + 1 == n_runs;
     TIMED(CLS_LINEAR, B200_TRY(linear<T>(h, hb, W, L.cat, proj, L.ldp, n_tok)));
     const bool diff = L.c.mixer == B200_MIXER_DIFF_ATTENTION;
     if (L.nsmall) TIMED(CLS_FOLD, B200_TRY(small_proj<T>(h, hb, W, L.w_small, nullptr, h->small32, n_tok, L.nsmall, W)));
-    const int Rv = diff ? L.ob_ld : a.heads * a.vdim;
+    const int Rv = L.ob_ld ? L.ob_ld : a.heads * a.vdim;
     if (diff) {
-      B200_TRY(diff_attention<T>(h, L, n_tok, max_ctx));
+      B200_TRY((map_attention<T, 2>(h, L, n_tok, max_ctx)));
+    } else if (L.c.mixer == B200_MIXER_BIAS_ATTENTION) {
+      B200_TRY((map_attention<T, 1>(h, L, n_tok, max_ctx)));
+    } else if (L.c.mixer == B200_MIXER_LATENT_ATTENTION) {
+      B200_TRY(joint_latent_attention<T>(h, L, n_tok, max_ctx));
+    } else if (L.c.mixer == B200_MIXER_RGLRU) {
+      B200_TRY(rglru<T>(h, L, n_tok));
     } else if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) {
       const bool blend = a.v_mix && li != h->vmix_first, keep = a.v_mix && li == h->vmix_first;
       TIMED(CLS_ELEMENTWISE, B200_LAUNCH(attn_rope_cache_kernel<T>, n_tok, 256, (size_t)a.rot_dims * 4 + 4, st, proj, (long long)L.ldp, L.p_q, L.p_k, L.p_v, L.Nq, L.Nk, L.Nv,
@@ -1591,14 +1966,18 @@ int step_parallel(b200_dlm* h, int n_tok, int n_want, int max_ctx, float* logits
       TIMED(CLS_ELEMENTWISE, B200_LAUNCH(gated_gelu_kernel<T>, (unsigned)ceil_div64(n, 256), 256, 0, st, proj, (long long)L.ldp, L.p_ffg, L.p_ffu, act, L.c.ff, n));
       TIMED(CLS_LINEAR, B200_TRY(linear<T>(h, act, L.c.ff, L.down, static_cast<T*>(h->ffo), W, n_tok)));
       ffo = static_cast<const T*>(h->ffo);
-    } else if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU || L.c.mlp == B200_MLP_MOE_SILU_GLU) {
+    } else if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU || L.c.mlp == B200_MLP_MOE_SILU_GLU || L.c.mlp == B200_MLP_MOE_GELU) {
       TIMED(CLS_EXPERTS, B200_TRY(routed_experts_glu<T>(h, L, hb, n_tok)));
       yexp = static_cast<const T*>(h->yexp);
     }
-    auto block_end = n_tok <= 592 && W <= 4096 ? parallel_block_end_kernel<T, true> : parallel_block_end_kernel<T, false>;
-    TIMED(CLS_ELEMENTWISE, B200_LAUNCH(block_end, n_tok, 256, 0, st, h->xin, mixo, ffo, yexp, h->moe_w, L.c.top,
-                                       h->trace_layers ? h->trace + (long long)li * stride : nullptr, last ? nullptr : h->layers[li + 1].n1w, hb, W, c.norm_eps, c.norm == B200_NORM_LAYER,
-                                       L.c.identity > 0 ? h->moe_idx : (const int*)nullptr, L.c.experts));
+    const bool side = c.side_dim > 0, copy = side && n_tok > SIDE_FEW;      // the token input comes behind the sum: it reads the residual, or its rounding for many tokens
+    auto block_end = n_tok <= 592 && W <= 4096 && !copy ? parallel_block_end_kernel<T, true> : parallel_block_end_kernel<T, false>;
+    float* trace = h->trace_layers ? h->trace + (long long)li * stride : nullptr;
+    const float *step = last ? nullptr : h->layers[li + 1].step, *w_next = last ? nullptr : h->layers[li + 1].n1w;
+    TIMED(CLS_ELEMENTWISE, B200_LAUNCH(block_end, n_tok, 256, 0, st, h->xin, mixo, ffo, yexp, h->moe_w, L.c.top, side ? nullptr : trace, side ? nullptr : w_next, hb, W, c.norm_eps,
+                                       copy ? ROW_COPY : c.norm == B200_NORM_LAYER ? ROW_LAYER : ROW_RMS,
+                                       L.c.identity > 0 ? h->moe_idx : (const int*)nullptr, L.c.experts, side ? nullptr : step));
+    if (side) B200_TRY(token_input<T>(h, L, n_tok, trace, step, w_next));
   }
   B200_TRY(check_launch("decoder LM layers"));
   if (n_want > 0) {
@@ -1957,6 +2336,10 @@ int b200_dlm_create(const b200_dlm_config* cfg, b200_dlm** out) {
   if (cfg->block == B200_BLOCK_PRE_NORM_STREAMS && (cfg->streams < 0 || cfg->streams > B200_DLM_MAX_STREAMS))
     B200_FAIL(B200_ERR_INVALID, "dlm_create: streams must be in 0..%d", B200_DLM_MAX_STREAMS);
   if (cfg->tied_head && cfg->block != B200_BLOCK_PRE_NORM_STREAMS) B200_FAIL(B200_ERR_INVALID, "dlm_create: a tied head is registered for the pre-norm streams block only");
+  if ((cfg->side_dim || cfg->loop_times) && (cfg->block != B200_BLOCK_PARALLEL_RESIDUAL || cfg->norm != B200_NORM_RMS))
+    B200_FAIL(B200_ERR_INVALID, "dlm_create: the token input and the loop are registered for the parallel block on a plain RMS norm only");
+  if (cfg->side_dim < 0 || cfg->loop_times < 0 || (cfg->loop_times > 0 && (cfg->loop_start < 0 || cfg->loop_stop <= cfg->loop_start || cfg->loop_stop > cfg->n_layers)))
+    B200_FAIL(B200_ERR_INVALID, "dlm_create: side_dim must not be negative and a loop must name a stretch of the layers");
   if (cfg->canon_taps < 0 || cfg->canon_taps > 64) B200_FAIL(B200_ERR_INVALID, "dlm_create: canon_taps must be in 0..64");
   for (int i = 0; i < cfg->n_layers; ++i) {
     const b200_dlm_layer& l = cfg->layers[i];
@@ -1984,10 +2367,21 @@ int b200_dlm_create(const b200_dlm_config* cfg, b200_dlm** out) {
       if (l.mlp != B200_MLP_NONE && l.mlp != B200_MLP_DENSE_RELU2) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: mlp kind %d is not registered for this block arrangement", i, l.mlp);
     } else if (cfg->block == B200_BLOCK_PARALLEL_RESIDUAL) {
       if (a.heads < 1 || a.dim < 1 || a.vdim < 1) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: heads, dim and vdim must be positive", i);
-      if (a.rot_dims < 0 || a.rot_dims % 2 || a.rot_dims > a.dim) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: rot_dims must be even and at most dim", i);
+      if (a.rot_dims < 0 || a.rot_dims % 2 || (a.rot_dims > a.dim && l.mixer != B200_MIXER_LATENT_ATTENTION)) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: rot_dims must be even and at most dim", i);
       if (a.rot_dims > 0 && a.rot_scaling == B200_ROT_RAMP && (!(a.rot_factor > 0.f) || !(a.rot_original > 0.f) || !(a.rot_fast > 0.f) || !(a.rot_slow > 0.f) || !(a.rot_base > 1.f)))
         B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: the rotary ramp wants positive factor, original, fast and slow", i);
-      if (l.mixer == B200_MIXER_SIGMOID_ATTENTION) {
+      const bool joint = l.mixer == B200_MIXER_LATENT_ATTENTION || l.mixer == B200_MIXER_BIAS_ATTENTION || l.mixer == B200_MIXER_RGLRU;
+      if (joint != (cfg->norm == B200_NORM_RMS)) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: mixer %d is not registered for this block's norm", i, l.mixer);
+      if (l.mixer == B200_MIXER_LATENT_ATTENTION) {
+        if (a.kv_rank < 1 || a.q_rank < 0 || (a.kv_rank + a.rot_dims + 7) / 8 * 8 > 1024) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: kv_rank + rot_dims in 1..1024 and no negative q_rank", i);
+        if (a.head_gate || a.window < 0) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: the gate of this block's latent attention is element by element", i);
+      } else if (l.mixer == B200_MIXER_BIAS_ATTENTION) {
+        if (a.kv_heads < 1 || a.heads % a.kv_heads || a.rot_dims || a.chunk || a.kv_from >= 0 || !(a.bias_max > 0.f))
+          B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: attention with a distance bias wants heads a multiple of kv_heads, a positive bias_max and no rotation", i);
+      } else if (l.mixer == B200_MIXER_RGLRU) {
+        if (a.heads != 1 || a.vdim != a.dim || a.blocks < 1 || a.dim % a.blocks || a.conv_taps < 1 || a.conv_taps > 64)
+          B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: the RG-LRU wants one head of dim = vdim channels in equal blocks and conv_taps in 1..64", i);
+      } else if (l.mixer == B200_MIXER_SIGMOID_ATTENTION) {
         if (a.kv_heads < 1 || a.heads % a.kv_heads) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: attention wants heads a multiple of kv_heads", i);
       } else if (l.mixer == B200_MIXER_DIFF_ATTENTION) {
         if (a.kv_heads < 1 || a.heads % a.kv_heads || a.chunk < 0) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: attention wants heads a multiple of kv_heads and no negative chunk", i);
@@ -2008,12 +2402,13 @@ int b200_dlm_create(const b200_dlm_config* cfg, b200_dlm** out) {
         B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: mixer %d is not registered for this block arrangement", i, l.mixer);
       }
       const bool diff = l.mixer == B200_MIXER_DIFF_ATTENTION;
-      if (l.mlp != B200_MLP_NONE && (diff ? l.mlp != B200_MLP_DENSE_CLAMPED_GLU && l.mlp != B200_MLP_MOE_SILU_GLU : l.mlp != B200_MLP_DENSE_GATED_GELU && l.mlp != B200_MLP_MOE_CLAMPED_GLU))
+      if (l.mlp != B200_MLP_NONE && (joint ? l.mlp != B200_MLP_DENSE_SILU_GLU && l.mlp != B200_MLP_MOE_GELU : diff ? l.mlp != B200_MLP_DENSE_CLAMPED_GLU && l.mlp != B200_MLP_MOE_SILU_GLU : l.mlp != B200_MLP_DENSE_GATED_GELU && l.mlp != B200_MLP_MOE_CLAMPED_GLU))
         B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: mlp kind %d is not registered for this block arrangement", i, l.mlp);
       if (l.mlp == B200_MLP_MOE_CLAMPED_GLU && (l.experts < 1 || l.experts > 4096 || l.top < 1 || l.top > l.experts || l.top > 32 || !(l.expert_limit > 0.f)))
         B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: experts in 1..4096, top in 1..min(experts, 32) and a positive limit", i);
       if (l.mlp == B200_MLP_DENSE_CLAMPED_GLU && !(l.expert_limit > 0.f)) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: the gated unit wants a positive limit", i);
-      if (l.mlp == B200_MLP_MOE_SILU_GLU) {
+      if (l.mlp == B200_MLP_MOE_GELU && l.identity) B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: these experts have no identity ones beside them", i);
+      if (l.mlp == B200_MLP_MOE_SILU_GLU || l.mlp == B200_MLP_MOE_GELU) {
         const int n = l.experts + l.identity, groups = l.groups > 1 ? l.groups : 1, keep = groups > 1 ? l.groups_keep : 1;
         if (l.experts < 1 || l.identity < 0 || l.shared_ff < 0 || n > 4096 || n % groups || keep < 1 || keep > groups || l.top < 1 || l.top > n / groups * keep || l.top > 32)
           B200_FAIL(B200_ERR_INVALID, "dlm_create: layer %d: experts + identity in 1..4096, equal groups, and top in 1..32 within the kept groups", i);
@@ -2051,6 +2446,7 @@ int b200_dlm_create(const b200_dlm_config* cfg, b200_dlm** out) {
   for (int i = 0; i < cfg->n_layers; ++i) {
     Layer& L = h->layers[i];
     L.c = cfg->layers[i];
+    L.index = i;
     if (L.c.a.decay) L.decay.assign(L.c.a.decay, L.c.a.decay + L.c.a.heads);      // the caller's array does not outlive this call
     L.c.a.decay = L.c.b.decay = nullptr;
   }
@@ -2116,7 +2512,27 @@ int b200_dlm_finalize(b200_dlm* h) {
   }
   if (parallel) {
     h->vmix_first = -1;
-    for (int i = 0; i < c.n_layers; ++i) B200_TRY(finalize_parallel_layer(h, i, drop));
+    if (c.side_dim > 0) {
+      h->side_ld = (c.side_dim + 7) / 8 * 8; h->side_cols = c.n_layers * c.side_dim;
+      B200_TRY(matrix("side.embed", c.vocab, h->side_cols, &h->side_embed));      // gathered, like the embedding
+    }
+    for (int i = 0; i < c.n_layers; ++i) {
+      const int64_t before = h->weight_bytes;
+      B200_TRY(finalize_parallel_layer(h, i, drop));
+      h->layers[i].wbytes = h->weight_bytes - before;
+    }
+    if (c.loop_times > 0) {      // the layers in the order a token runs through them; a pass shares the weights
+      B200_TRY(get_f32_shaped(h, "loop.step", {c.loop_times, W}, &h->loop_step));
+      std::vector<Layer> runs(h->layers.begin(), h->layers.begin() + c.loop_start);
+      for (int t = 0; t < c.loop_times; ++t)
+        for (int i = c.loop_start; i < c.loop_stop; ++i) {
+          runs.push_back(h->layers[i]);
+          runs.back().repeat = t > 0;
+          if (i == c.loop_start) runs.back().step = h->loop_step + (size_t)t * W;
+        }
+      runs.insert(runs.end(), h->layers.begin() + c.loop_stop, h->layers.end());
+      h->layers = std::move(runs);
+    }
   }
   for (int i = 0; i < c.n_layers && !sandwich && !parallel && !streams; ++i) {
     Layer& L = h->layers[i];
@@ -2238,7 +2654,7 @@ int b200_dlm_cache_begin(b200_dlm* h, int slots, int capacity, int max_step_toke
   h->stream = static_cast<cudaStream_t>(stream);
   const bool sandwich = c.block == B200_BLOCK_SANDWICH, parallel = c.block == B200_BLOCK_PARALLEL_RESIDUAL, streams = c.block == B200_BLOCK_PRE_NORM_STREAMS;
   size_t max_ldp = 0, max_hr = 0, max_hv = 0, max_ff = 1, max_r = 0, max_tiles = 0, max_qkv = 1, max_rv = 1, max_gate = 1, max_e = 1, max_top = 0, max_part = 0, max_prep = 4, max_segrow = 1, max_heads = 1;
-  size_t max_small = 1, max_eff = 0, max_nv = 1;
+  size_t max_small = 1, max_eff = 0, max_nv = 1, max_qrank = 0, max_q2 = 0;
   for (auto& L : h->layers) {
     const b200_dlm_mixer &a = L.c.a, &b = L.c.b;
     max_ldp = std::max(max_ldp, (size_t)L.ldp);
@@ -2280,6 +2696,25 @@ int b200_dlm_cache_begin(b200_dlm* h, int slots, int capacity, int max_step_toke
         max_qkv = std::max(max_qkv, (size_t)L.Nq);
         max_hv = std::max(max_hv, (size_t)L.ob_ld);
         max_part = std::max(max_part, (size_t)(L.sig_mma >= 0 ? 64 : L.QT) * (2 * a.vdim + 4));
+      } else if (L.c.mixer == B200_MIXER_LATENT_ATTENTION) {
+        B200_TRY(A.alloc(&L.cache, (size_t)slots * capacity * L.rp * es));
+        max_hr = std::max(max_hr, (size_t)a.heads * L.rp);
+        max_qrank = std::max(max_qrank, (size_t)(a.q_rank + 7) / 8 * 8);
+        max_q2 = std::max(max_q2, (size_t)(L.Nq + 7) / 8 * 8);
+        max_hv = std::max(max_hv, (size_t)L.ob_ld);
+        max_part = std::max(max_part, (size_t)16 * (L.rp + 2));
+      } else if (L.c.mixer == B200_MIXER_BIAS_ATTENTION) {
+        B200_TRY(A.alloc(&L.kcache, (size_t)slots * capacity * L.Nk * es));
+        B200_TRY(A.alloc(&L.vcache, (size_t)slots * capacity * L.Nv * es));
+        max_qkv = std::max(max_qkv, (size_t)L.Nq);
+        max_hv = std::max(max_hv, (size_t)L.ob_ld);
+        max_part = std::max(max_part, (size_t)(L.sig_mma >= 0 ? 64 : L.QT) * (a.vdim + 2));
+      } else if (L.c.mixer == B200_MIXER_RGLRU) {
+        B200_TRY(A.alloc_t(&L.gru, (size_t)slots * a.dim));
+        if (a.conv_taps > 1) B200_TRY(A.alloc_t(&L.qkv_hist, (size_t)slots * (a.conv_taps - 1) * a.dim));
+        max_qkv = std::max(max_qkv, (size_t)a.dim);
+        max_gate = std::max(max_gate, (size_t)2 * a.dim);
+        max_hv = std::max(max_hv, (size_t)L.ob_ld);
       } else if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) {
         B200_TRY(A.alloc(&L.kcache, (size_t)slots * capacity * L.Nk * es));
         B200_TRY(A.alloc(&L.vcache, (size_t)slots * capacity * L.Nv * es));
@@ -2299,7 +2734,7 @@ int b200_dlm_cache_begin(b200_dlm* h, int slots, int capacity, int max_step_toke
         max_segrow = std::max(max_segrow, (size_t)a.heads * (a.vdim + 1) * a.dim);
         max_heads = std::max(max_heads, (size_t)a.heads);
       }
-      if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU || L.c.mlp == B200_MLP_MOE_SILU_GLU) {
+      if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU || L.c.mlp == B200_MLP_MOE_SILU_GLU || L.c.mlp == B200_MLP_MOE_GELU) {
         max_e = std::max(max_e, (size_t)L.c.experts); max_top = std::max(max_top, (size_t)L.c.top);
         max_eff = std::max(max_eff, (size_t)L.c.top * L.c.ff);
       }
@@ -2385,6 +2820,13 @@ int b200_dlm_cache_begin(b200_dlm* h, int slots, int capacity, int max_step_toke
     B200_TRY(A.alloc_t(&h->gate32, T * max_gate));
     B200_TRY(A.alloc(&h->ffo, T * W * es));
     B200_TRY(A.alloc(&h->vfirst, T * max_nv * es));
+    if (max_hr) {      // latent attention: query latents, queries, folded queries and weighted sums
+      B200_TRY(A.alloc(&h->cq, T * std::max(max_qrank, (size_t)1) * es));
+      B200_TRY(A.alloc(&h->q2, T * std::max(max_q2, (size_t)1) * es));
+      B200_TRY(A.alloc_t(&h->qa, T * max_hr));
+      B200_TRY(A.alloc_t(&h->ol, T * max_hr));
+    }
+    if (c.side_dim > 0) B200_TRY(A.alloc(&h->sidez, T * h->side_ld * es));
     h->part_floats = (size_t)600 * std::max(max_part, (size_t)1);
     if (max_top) {
       const size_t pairs = T * max_top, tiles = pairs / 64 + max_e + 2;
@@ -2440,7 +2882,7 @@ int b200_dlm_cache_begin(b200_dlm* h, int slots, int capacity, int max_step_toke
       max_ff *= max_top;        // the experts' hidden rows: one per (token, chosen expert)
     }
   }
-  if (h->trace_layers) B200_TRY(A.alloc_t(&h->trace, (size_t)c.n_layers * T * W));
+  if (h->trace_layers) B200_TRY(A.alloc_t(&h->trace, h->layers.size() * T * W));
   B200_TRY(A.alloc_t(&h->part, h->part_floats));
   B200_TRY(A.alloc(&h->hbuf, T * W * es));
   B200_TRY(A.alloc(&h->proj, T * max_ldp * es));
@@ -2640,11 +3082,11 @@ int b200_dlm_read_buffer(b200_dlm* h, const char* name, void* dst_dev, int64_t c
   if (n == "layers") {
     if (!h->trace) B200_FAIL(B200_ERR_STATE, "dlm_read_buffer: 'layers' needs option trace_layers = 1 before cache_begin");
     const int64_t row = (int64_t)h->last_tokens * W * 4;
-    const int64_t bytes = row * h->cfg.n_layers;
+    const int64_t bytes = row * (int64_t)h->layers.size();
     if (nbytes) *nbytes = bytes;
     if (!dst_dev) return B200_OK;
     if (capacity_bytes < bytes) B200_FAIL(B200_ERR_SHAPE, "dlm_read_buffer: '%s' needs %lld bytes", name, (long long)bytes);
-    B200_CUDA(cudaMemcpy2DAsync(dst_dev, (size_t)row, h->trace, (size_t)h->tmax * W * 4, (size_t)row, (size_t)h->cfg.n_layers,
+    B200_CUDA(cudaMemcpy2DAsync(dst_dev, (size_t)row, h->trace, (size_t)h->tmax * W * 4, (size_t)row, h->layers.size(),
                                 cudaMemcpyDeviceToDevice, h->stream));
     return B200_OK;
   }
@@ -2687,16 +3129,21 @@ int64_t b200_dlm_algorithmic_bytes(b200_dlm* h, int tokens, int context) {
   if (h->cfg.block == B200_BLOCK_PARALLEL_RESIDUAL) {      // `tokens` = requests when decoding, as for the sandwich block
     for (auto& L : h->layers) {
       const b200_dlm_mixer& a = L.c.a;
-      if (L.c.mixer == B200_MIXER_DIFF_ATTENTION) {      // every request reads its chunk up to its own position, and writes a row where the layer owns the cache
+      if (L.repeat) b += L.wbytes;      // a further pass reads the weights again
+      if (L.c.mixer == B200_MIXER_LATENT_ATTENTION) b += ((int64_t)context + tokens) * L.rp * es;
+      else if (L.c.mixer == B200_MIXER_RGLRU) b += 2 * (int64_t)tokens * a.dim * 4 * a.conv_taps;      // the state and the carried inputs, read and written
+      else if (L.c.mixer == B200_MIXER_BIAS_ATTENTION) b += ((int64_t)context + tokens) * (L.Nk + L.Nv) * es;
+      else if (L.c.mixer == B200_MIXER_DIFF_ATTENTION) {      // every request reads its chunk up to its own position, and writes a row where the layer owns the cache
         const int64_t per = tokens > 0 ? (int64_t)context / tokens : 0, seen = a.chunk > 0 ? per % a.chunk : per;
         b += (seen + (a.kv_from < 0 ? 1 : 0)) * tokens * (L.Nk + L.Nv) * es;
       } else if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) b += ((int64_t)context + tokens) * (L.Nk + L.Nv) * es;      // every cached key and value once
       else b += 2 * (int64_t)tokens * a.heads * a.dim * a.vdim * 4;                                              // the matrix memories, read and written
-      if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU || L.c.mlp == B200_MLP_MOE_SILU_GLU) {
+      if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU || L.c.mlp == B200_MLP_MOE_SILU_GLU || L.c.mlp == B200_MLP_MOE_GELU) {
         const int64_t used = std::min<int64_t>(L.c.experts, (int64_t)tokens * L.c.top);
-        b -= (int64_t)(L.c.experts - used) * 3 * L.c.ff * W * es;
+        b -= (int64_t)(L.c.experts - used) * (L.c.mlp == B200_MLP_MOE_GELU ? 2 : 3) * L.c.ff * W * es;
       }
     }
+    b += (int64_t)tokens * h->side_cols * es;      // the tokens' rows of the second table
     return b + (int64_t)tokens * W * es;
   }
   if (h->cfg.block != B200_BLOCK_SANDWICH) {
@@ -2738,14 +3185,18 @@ int64_t b200_dlm_algorithmic_flops(b200_dlm* h, int tokens, int context) {
     }
     if (h->cfg.block == B200_BLOCK_PARALLEL_RESIDUAL) {
       const b200_dlm_mixer& a = L.c.a;
-      f += 2 * T * W * L.ncat + 2 * T * W * L.nsmall + 2 * T * W * (L.c.mixer == B200_MIXER_DIFF_ATTENTION ? L.ob_ld : a.heads * a.vdim);
-      if (L.c.mixer == B200_MIXER_DIFF_ATTENTION) {
+      f += 2 * T * W * L.ncat + 2 * T * W * L.nsmall + 2 * T * W * (L.ob_ld ? L.ob_ld : a.heads * a.vdim) + 4 * T * W * h->cfg.side_dim;
+      if (L.c.mixer == B200_MIXER_LATENT_ATTENTION) f += 2 * T * (int64_t)L.Nq * a.q_rank + 2 * T * a.heads * (a.dim + a.vdim) * a.kv_rank + 4 * (T * context + T * (T + 1) / 2) * a.heads * (a.kv_rank + a.rot_dims);
+      else if (L.c.mixer == B200_MIXER_BIAS_ATTENTION) f += 2 * (T * context + T * (T + 1) / 2) * a.heads * (a.dim + a.vdim);
+      else if (L.c.mixer == B200_MIXER_RGLRU) f += 4 * T * a.dim * (a.dim / a.blocks);
+      else if (L.c.mixer == B200_MIXER_DIFF_ATTENTION) {
         int64_t pairs = 0;       // (query, key) pairs of one prompt of T tokens on top of `context`
         for (int64_t t = 0; t < T; ++t) pairs += (a.chunk > 0 ? (context + t) % a.chunk : context + t) + 1;
         f += 4 * pairs * a.heads * (a.dim + a.vdim);
       } else if (L.c.mixer == B200_MIXER_SIGMOID_ATTENTION) f += 2 * a.heads * (a.dim + a.vdim + a.heads) * (T * context + T * (T + 1) / 2);      // scores, head mix, sums
       else f += (L.c.mixer == B200_MIXER_DELTA ? 8 : 4) * T * a.heads * a.dim * a.vdim;
       if (L.c.mlp == B200_MLP_DENSE_GATED_GELU) f += 2 * T * W * L.c.ff;                   // the down-projection (gate and value are inside ncat)
+      if (L.c.mlp == B200_MLP_MOE_GELU) f += 4 * T * L.c.top * W * L.c.ff;
       if (L.c.mlp == B200_MLP_MOE_CLAMPED_GLU || L.c.mlp == B200_MLP_MOE_SILU_GLU) f += 6 * T * L.c.top * W * L.c.ff;
       continue;
     }

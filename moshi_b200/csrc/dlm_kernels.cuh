@@ -133,17 +133,19 @@ __global__ void __launch_bounds__(256) relu2_kernel(const T* __restrict__ proj, 
 // C[z][M][N] = alpha * A[z][M][K] . B[z][N][K]^T on the CUDA cores (fp32 FMA; inputs converted on load): the all-fp32 mode's
 // linear, the per-head products around the latent attention, and the bf16 mode's linear for shapes the tcgen05 GEMM does not take.
 // A row's sum runs over k in order whatever M is: a token's result does not depend on what else is in the step.
-// accumulate: C += instead of C =.
+// accumulate: C += instead of C =.  gate (TC rows of ldg elements, sg per batch): C times sigmoid(gate) element by element.
 template <typename TA, typename TB, typename TC>
 __global__ void __launch_bounds__(256) gemm_nt_kernel(const TA* __restrict__ A, long long lda, long long sa, const TB* __restrict__ B,
                                                       long long ldb, long long sb, TC* __restrict__ C, long long ldc, long long sc,
                                                       int M, int N, int K, float alpha, int accumulate = 0, int zdiv = 0,
-                                                      long long sa2 = 0, long long sb2 = 0, long long sc2 = 0) {
+                                                      long long sa2 = 0, long long sb2 = 0, long long sc2 = 0, const TC* __restrict__ gate = nullptr,
+                                                      long long ldg = 0, long long sg = 0) {
   constexpr int BM = 64, BN = 64, BK = 16;
   __shared__ float As[BK][BM + 1], Bs[BK][BN + 1];
   {   // batch index z, or (z / zdiv, z % zdiv) with strides of their own for the outer index (zdiv > 0)
     const long long z1 = zdiv > 0 ? blockIdx.z % zdiv : blockIdx.z, z2 = zdiv > 0 ? blockIdx.z / zdiv : 0;
     A += z1 * sa + z2 * sa2; B += z1 * sb + z2 * sb2; C += z1 * sc + z2 * sc2;
+    if (gate) gate += z1 * sg;
   }
   const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -173,7 +175,11 @@ __global__ void __launch_bounds__(256) gemm_nt_kernel(const TA* __restrict__ A, 
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int m = m0 + ty + 16 * i, n = n0 + tx + 16 * j;
-      if (m < M && n < N) C[(long long)m * ldc + n] = from_f<TC>(alpha * acc[i][j] + (accumulate ? to_f(C[(long long)m * ldc + n]) : 0.f));
+      if (m < M && n < N) {
+        float v = alpha * acc[i][j] + (accumulate ? to_f(C[(long long)m * ldc + n]) : 0.f);
+        if (gate) v *= sigmoidf(to_f(gate[(long long)m * ldg + n]));
+        C[(long long)m * ldc + n] = from_f<TC>(v);
+      }
     }
 }
 
@@ -657,15 +663,17 @@ __global__ void __launch_bounds__(128) latent_attn_merge_kernel(const float* __r
 // C[z][M][N] = alpha * A[z][M][K] . B[z][N][K]^T on the tensor cores (mma.sync m16n8k16, bf16 in, fp32 accumulate) for the
 // per-head products around the latent attention in bfloat16: A is bf16 or fp32 (rounded to bf16 on its way into shared
 // memory), B bf16, C fp32 or bf16.  K a multiple of 16; M and N are free (zero-filled edges).  CTA tile 64 x 64, 4 warps of
-// 16 rows x 64 columns, 32-element k-steps through shared memory.
+// 16 rows x 64 columns, 32-element k-steps through shared memory.  gate: as in gemm_nt_kernel.
 template <typename TA, typename TC>
 __global__ void __launch_bounds__(128) gemm_nt_mma_kernel(const TA* __restrict__ A, long long lda, long long sa, const bf16* __restrict__ B,
                                                           long long ldb, long long sb, TC* __restrict__ C, long long ldc, long long sc,
-                                                          int M, int N, int K, float alpha) {
+                                                          int M, int N, int K, float alpha, const TC* __restrict__ gate = nullptr,
+                                                          long long ldg = 0, long long sg = 0) {
   constexpr int BM = 64, BN = 64, BK = 32, ST = BK + 8;
   __shared__ __align__(16) bf16 As[BM][ST];
   __shared__ __align__(16) bf16 Bs[BN][ST];
   A += (long long)blockIdx.z * sa; B += (long long)blockIdx.z * sb; C += (long long)blockIdx.z * sc;
+  if (gate) gate += (long long)blockIdx.z * sg;
   const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
   float acc[8][4];
@@ -730,8 +738,9 @@ __global__ void __launch_bounds__(128) gemm_nt_mma_kernel(const TA* __restrict__
     for (int hf = 0; hf < 2; ++hf) {
       const int m = m0 + warp * 16 + g + 8 * hf, n = n0 + nb * 8 + 2 * t4;
       if (m < M) {
-        if (n < N) C[(long long)m * ldc + n] = from_f<TC>(alpha * acc[nb][2 * hf]);
-        if (n + 1 < N) C[(long long)m * ldc + n + 1] = from_f<TC>(alpha * acc[nb][2 * hf + 1]);
+        auto gated = [&](float v, int col) { return from_f<TC>(gate ? v * sigmoidf(to_f(gate[(long long)m * ldg + col])) : v); };
+        if (n < N) C[(long long)m * ldc + n] = gated(alpha * acc[nb][2 * hf], n);
+        if (n + 1 < N) C[(long long)m * ldc + n + 1] = gated(alpha * acc[nb][2 * hf + 1], n + 1);
       }
     }
 }

@@ -86,11 +86,11 @@ __global__ void __launch_bounds__(256) causal_conv_kernel(const TI* __restrict__
 template <typename TI>
 __global__ void __launch_bounds__(256) conv_carry_kernel(const TI* __restrict__ in, long long ld_in, float* __restrict__ hist, int C, int keep,
                                                          const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
-                                                         const int* __restrict__ tok_last) {
+                                                         const int* __restrict__ tok_last, const float* __restrict__ bias = nullptr) {      // bias: added to the inputs
   const long long t = blockIdx.x;
   if (tok_last[t] - (int)t >= keep) return;                // not among the request's last taps - 1 tokens of this step
   float* dst = hist + ((long long)tok_slot[t] * keep + tok_pos[t] % keep) * C;
-  for (int c = threadIdx.x; c < C; c += blockDim.x) dst[c] = to_f(in[t * ld_in + c]);
+  for (int c = threadIdx.x; c < C; c += blockDim.x) dst[c] = to_f(in[t * ld_in + c]) + (bias ? bias[c] : 0.f);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
@@ -1129,7 +1129,8 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int* __restrict__
 }
 
 // Grouped product of the routed experts: for tile (expert e, rows pos0 .. pos0 + n - 1 of the grouped order)
-//   C[c_rows ? c_rows[pos] : pos][:] = act( A[a_rows ? a_rows[pos] : pos][:] . B[e]^T ),  B[e] = B + e * sb, [N][K];  act 1: relu(.)^2
+//   C[c_rows ? c_rows[pos] : pos][:] = act( A[a_rows ? a_rows[pos] : pos][:] . B[e]^T ),  B[e] = B + e * sb, [N][K];  act 1: relu(.)^2,
+// act 4: erf GELU
 // CUDA cores, fp32 FMA, k in order (the all-fp32 mode, and shapes the tensor-core kernel does not take).
 template <typename TA, typename TB, typename TC>
 __global__ void __launch_bounds__(256) grouped_gemm_kernel(const TA* __restrict__ A, long long lda, const int* __restrict__ a_rows,
@@ -1175,7 +1176,8 @@ __global__ void __launch_bounds__(256) grouped_gemm_kernel(const TA* __restrict_
       const int m = ty + 16 * i, n = n0 + tx + 16 * j;
       if (m < M && n < N) {
         float v = acc[i][j];
-        if (act) { v = fmaxf(v, 0.f); v = v * v; }
+        if (act == 4) v = 0.5f * v * (1.f + erff(v * 0.7071067811865476f));
+        else if (act) { v = fmaxf(v, 0.f); v = v * v; }
         const long long crow = c_rows ? c_rows[pos0 + m] : pos0 + m;
         C[crow * ldc + n] = from_f<TC>(v);
       }
@@ -1184,7 +1186,8 @@ __global__ void __launch_bounds__(256) grouped_gemm_kernel(const TA* __restrict_
 
 // The same grouped product on the tensor cores (mma.sync m16n8k16, bf16 in, fp32 accumulate): K a multiple of 16, rows of A
 // and B on 16-byte boundaries; act 2: gate and value rows of B alternate and the epilogue writes
-// min(g, limit) * sigmoid(1.702 min(g, limit)) * (clamp(u, -limit, limit) + 1) into column n / 2, act 3 silu(g) * u.  CTA tile 128 x 128 (tiles of 128 rows in the tile table), 8 warps of 32 x 64, 64-element
+// min(g, limit) * sigmoid(1.702 min(g, limit)) * (clamp(u, -limit, limit) + 1) into column n / 2, act 3 silu(g) * u;
+// act 4: erf GELU of every column.  CTA tile 128 x 128 (tiles of 128 rows in the tile table), 8 warps of 32 x 64, 64-element
 // k-steps through two shared-memory buffers filled by cp.async (chunks outside M, N or K are zero-filled by a copy of size 0).
 __device__ __forceinline__ void cp_async_16_or_zero(void* smem_dst, const void* src, bool valid) {
   const unsigned d = (unsigned)__cvta_generic_to_shared(smem_dst);
@@ -1265,7 +1268,7 @@ __global__ void __launch_bounds__(256, 2) grouped_gemm_mma_kernel(const bf16* __
       for (int nb = 0; nb < 8; ++nb) {
         const int n = n0 + wn + nb * 8 + 2 * t4;
         float v0 = acc[mf][nb][2 * hf], v1 = acc[mf][nb][2 * hf + 1];
-        if (act >= 2) {      // rows of B interleave gate and value: columns (n, n + 1) are one output, column n / 2 of C
+        if (act == 2 || act == 3) {      // rows of B interleave gate and value: columns (n, n + 1) are one output, column n / 2 of C
           if (n + 1 < N && act == 3) {
             C[crow * ldc + (n >> 1)] = __float2bfloat16_rn(v0 / (1.f + expf(-v0)) * v1);
           } else if (n + 1 < N) {
@@ -1274,7 +1277,8 @@ __global__ void __launch_bounds__(256, 2) grouped_gemm_mma_kernel(const bf16* __
           }
           continue;
         }
-        if (act) { v0 = fmaxf(v0, 0.f); v0 *= v0; v1 = fmaxf(v1, 0.f); v1 *= v1; }
+        if (act == 4) { v0 = 0.5f * v0 * (1.f + erff(v0 * 0.7071067811865476f)); v1 = 0.5f * v1 * (1.f + erff(v1 * 0.7071067811865476f)); }
+        else if (act) { v0 = fmaxf(v0, 0.f); v0 *= v0; v1 = fmaxf(v1, 0.f); v1 *= v1; }
         if (n + 1 < N && pair_ok) {
           *reinterpret_cast<unsigned*>(C + crow * ldc + n) = pack_bf16(v0, v1);
         } else {

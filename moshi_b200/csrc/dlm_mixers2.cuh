@@ -21,19 +21,24 @@ __device__ __forceinline__ float clamped_gluf(float g, float u, float limit) {
   return g * sigmoidf(1.702f * g) * (u + 1.f);
 }
 
-// the block's norm of one fp32 row -> T: layer norm without a bias, or RMS norm (w = 1 + the stored weight)
+// the block's norm of one fp32 row -> T (`layer`): ROW_RMS (w as it is multiplied), ROW_LAYER without a bias, ROW_COPY: the row itself
+enum { ROW_RMS = 0, ROW_LAYER = 1, ROW_COPY = 2 };
 template <typename T>
 __device__ __forceinline__ void block_norm(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ h, int W, float eps, int layer, float* red) {
-  if (layer) { block_layernorm<T>(x, w, nullptr, h, W, eps, red); return; }
+  if (layer == ROW_COPY) {
+    for (int i = threadIdx.x; i < W; i += blockDim.x) h[i] = from_f<T>(x[i]);
+    return;
+  }
+  if (layer == ROW_LAYER) { block_layernorm<T>(x, w, nullptr, h, W, eps, red); return; }
   const float r = block_rrms(x, W, eps, red);
   for (int i = threadIdx.x; i < W; i += blockDim.x) h[i] = from_f<T>(x[i] * r * w[i]);
 }
 
-// x = table[token] * scale -> residual stream (fp32);  h = norm(x) * w1 -> T
+// x = table[token] * scale (+ step: the vector in front of a pass) -> residual stream (fp32);  h = norm(x) * w1 -> T
 template <typename T>
 __global__ void __launch_bounds__(256) embed_scale_norm_kernel(const int* __restrict__ tokens, const T* __restrict__ table, int vocab, int W, float scale,
                                                                const float* __restrict__ w1, float* __restrict__ xin, T* __restrict__ h, float eps,
-                                                               int* __restrict__ err, int layer) {
+                                                               int* __restrict__ err, int layer, const float* __restrict__ step = nullptr) {
   __shared__ float red[32];
   const long long t = blockIdx.x;
   int id = tokens[t];
@@ -41,21 +46,23 @@ __global__ void __launch_bounds__(256) embed_scale_norm_kernel(const int* __rest
   if (bad) { if (threadIdx.x == 0) atomicOr(err, ERR_TOKEN); id = 0; }
   const T* row = table + (long long)id * W;
   float* x = xin + t * W;
-  for (int i = threadIdx.x; i < W; i += blockDim.x) x[i] = bad ? 0.f : to_f(row[i]) * scale;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) x[i] = (bad ? 0.f : to_f(row[i]) * scale) + (step ? step[i] : 0.f);
   __syncthreads();
   block_norm<T>(x, w1, h + t * W, W, eps, layer, red);
 }
 
 // End of a parallel block, one CTA per token:  x <- x + mix + ff,  ff = a dense feed-forward's row | sum_k ew[t][k] * rows of
 // the chosen experts (the row of h itself for a choice from n_exp on: an identity expert) | both | nothing;  optional copy of x
-// (per-layer trace);  optional h = norm(x) * w_next for the next layer.
+// (per-layer trace);  x <- x + step (the vector in front of a pass, when given);  optional h = norm(x) * w_next for the next layer
+// (layer = ROW_COPY, not with REG: h = x as it is).
 // REG (few tokens, W <= 4096): the row stays in registers between the sum and the norm, which shortens the chain of a CTA; many tokens
 // fill the SMs better with the smaller kernel.
 template <typename T, bool REG>
 __global__ void __launch_bounds__(256) parallel_block_end_kernel(float* __restrict__ xin, const T* __restrict__ mix, const T* __restrict__ ff,
                                                                  const T* __restrict__ yexp, const float* __restrict__ ew, int top,
                                                                  float* __restrict__ trace, const float* __restrict__ w_next, T* h,
-                                                                 int W, float eps, int layer = 0, const int* __restrict__ choice = nullptr, int n_exp = 0) {
+                                                                 int W, float eps, int layer = 0, const int* __restrict__ choice = nullptr, int n_exp = 0,
+                                                                 const float* __restrict__ step = nullptr) {
   __shared__ float red[32];
   const long long t = blockIdx.x;
   float* x = xin + t * W;
@@ -84,8 +91,9 @@ __global__ void __launch_bounds__(256) parallel_block_end_kernel(float* __restri
     for (int k = 0; k < NR; ++k) {
       const int i = threadIdx.x + 256 * k;
       if (i >= W) break;
-      x[i] = v[k];
       if (trace) trace[t * W + i] = v[k];
+      if (step) v[k] += step[i];
+      x[i] = v[k];
       s += v[k];
     }
     if (!w_next) return;
@@ -103,11 +111,12 @@ __global__ void __launch_bounds__(256) parallel_block_end_kernel(float* __restri
     return;
   }
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
-    const float v = updated(i);
-    x[i] = v;
+    float v = updated(i);
     if (trace) trace[t * W + i] = v;
+    if (step) v += step[i];
+    x[i] = v;
   }
-  if (w_next) {
+  if (w_next || layer == ROW_COPY) {
     __syncthreads();
     block_norm<T>(x, w_next, h + t * W, W, eps, layer, red);
   }

@@ -29,6 +29,7 @@ def _fill_mixer(dst, m: MixerConfig) -> None:
     dst.softcap, dst.v_mix = m.softcap, int(m.v_mix)
     dst.bias, dst.sink, dst.head_gate = int(m.bias), SINKS[m.sink], int(m.head_gate)
     dst.chunk, dst.qk_norm, dst.diff, dst.kv_from = m.chunk, int(m.qk_norm), m.diff, m.kv_from
+    dst.q_rank, dst.out_gate, dst.bias_max, dst.q_temp_coef, dst.q_temp_every, dst.blocks = m.q_rank, int(m.out_gate), m.bias_max, m.q_temp_coef, m.q_temp_every, m.blocks
     if m.decay:
         dst.decay = (C.c_float * len(m.decay))(*m.decay)      # ctypes keeps the array alive with the struct; create() copies it
 
@@ -66,6 +67,7 @@ class DecoderLM:
         c.block, c.canon_taps, c.logit_softcap = BLOCKS[cfg.block], cfg.canon_taps, cfg.logit_softcap
         c.streams, c.logit_scale, c.tied_head = cfg.streams, cfg.logit_scale, int(cfg.tied_head)
         c.norm = NORMS[cfg.norm]
+        c.side_dim, c.loop_start, c.loop_stop, c.loop_times = cfg.side_dim, cfg.loop_start, cfg.loop_stop, cfg.loop_times
         c.compute_dtype = _DTYPES[dtype]
         c.layers = layers
         items = tensors.items() if isinstance(tensors, tp.Mapping) else tensors
@@ -197,8 +199,9 @@ class DecoderLMGen:
         return out
 
     def layer_outputs(self) -> torch.Tensor:
-        """What every layer handed on in the last step, f32 [layers, tokens, width] (needs ``trace_layers=True``)."""
-        return self.read_buffer("layers", torch.float32, (len(self.model.cfg.layers), self._last_tokens, self.model.width))
+        """What every layer handed on in the last step, f32 [layer runs, tokens, width] (a layer of a loop counts once per pass; needs
+        ``trace_layers=True``)."""
+        return self.read_buffer("layers", torch.float32, (len(self.model.cfg.layer_runs()), self._last_tokens, self.model.width))
 
     def error_flags(self) -> int:
         return int(self.read_buffer("error_flags", torch.int32, (1,)).item())

@@ -291,6 +291,12 @@ def iter_synth_decoder_tensors(cfg: DecoderLMConfig, seed: int = 99, device="cpu
             t = 0.3 + _uniform(gen, shape, 0.2, device)
         elif last == "pb":              # sigmoid weights are not normalised over keys: start them small
             t = -2.0 + _uniform(gen, shape, 0.5, device)
+        elif last == "lam":             # RG-LRU: from memories of a few tokens to memories of hundreds
+            t = -4.5 + _uniform(gen, shape, 2.0, device)
+        elif last == "rel":             # a bias by distance that matters beside the scores
+            t = _uniform(gen, shape, 1.0, device)
+        elif leaf == "loop.step":
+            t = _uniform(gen, shape, 0.5, device)
         elif last == "A_log":           # delta rule: decays near one
             t = -1.5 + _uniform(gen, shape, 0.5, device)
         elif last in ("dt_bias", "correction"):
@@ -310,7 +316,7 @@ def iter_synth_decoder_tensors(cfg: DecoderLMConfig, seed: int = 99, device="cpu
         elif leaf == "dwa":
             t = torch.rand(shape, generator=gen, device=device) + 0.2
             t = t / t.sum()
-        elif leaf == "embed":
+        elif leaf in ("embed", "side.embed"):
             t = _uniform(gen, shape, 1.0, device)
         else:
             t = _uniform(gen, shape, math.sqrt(3.0 / shape[-1]), device)
