@@ -1168,6 +1168,168 @@ def megolorn_arm(args) -> None:
     print(json.dumps(out))
 
 
+# ---------------------------------------------------------------------------------------------
+# --decoder-lm --decoder-arch korirax: the Korirax design, whole and one mechanism at a time, beside the like kernels of the existing
+# designs at equal shapes (Dibulix: latent attention with a rotated part, minGRU; Megolorn: attention, gated units, experts; and a
+# Megolorn model of equal width, depth, projection sizes and feed-forwards as the closest whole model)
+# ---------------------------------------------------------------------------------------------
+KORIRAX_SIZES = {
+    # name: (width, layer kinds, heads, kv heads, head dim, rotated dims, kv_rank, q_rank, recurrence width, blocks, experts, top, expert ff, shared ff, dense ff, token input, vocab)
+    "w2048": (2048, ("latent_attention", "attention", "rglru", "attention"), 16, 4, 128, 64, 512, 768, 2048, 16, 16, 2, 4096, 4096, 8192, 256, 32000),
+    "w4096": (4096, ("latent_attention", "attention", "rglru"), 16, 4, 128, 64, 512, 1536, 4096, 16, 16, 2, 8192, 8192, 16384, 256, 32000),
+}
+
+
+def _korirax_cfgs(size: str) -> dict:
+    """name -> configuration: the whole model, small models of one mechanism each, and the comparators."""
+    from moshi_b200.config import DecoderLMConfig
+    W, kinds, H, G, d, rd, r, qr, N, nb, E, top, ff, sff, dff, side, V = KORIRAX_SIZES[size]
+    ramp = {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}
+    mix = {"latent_attention": {"dim": d, "heads": H, "kv_rank": r, "q_rank": qr, "rot_dim": rd, "rot": {"base": 1e5, "dims": rd, "scaling": ramp}, "scale": (d + rd) ** -0.5, "vdim": d},
+           "attention": {"bias_max": 512, "dim": d, "heads": H, "kv_heads": G, "q_temp": {"coef": 0.1, "every": 4096}, "scale": d ** -0.5, "vdim": d},
+           "rglru": {"blocks": nb, "conv": 4, "width": N}}
+    dense = {"ff": dff, "kind": "dense"}
+    moe = {"expert": {"ff": ff}, "kind": "moe", "router": {"experts": E, "groups": {"count": 4, "keep": 2}, "scale": 2.0, "top": top}, "shared": {"ff": sff}}
+
+    def kor(layers, side=0, loop=None):
+        c = {"architecture": "Korirax", "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "vocab": V, "width": W, "layers": [{"type": k, "mixer": mix[k], "mlp": m} for k, m in layers]}
+        if side:
+            c["token_side"] = {"dim": side}
+        if loop:
+            c["loop"] = dict(zip(("start", "stop", "times"), loop))
+        return DecoderLMConfig.from_dict(c)
+
+    # the comparator's gated experts have three matrices, this design's two: equal bytes per expert
+    glu = lambda f: f * 2 // 3 // 64 * 64
+    meg_mix = {"diff": 0.5, "dim": d // 2, "heads": H, "kv_heads": G, "scale": (d // 2) ** -0.5, "vdim": d}
+    meg_moe = {"expert": {"ff": glu(ff)}, "kind": "moe", "router": {"experts": E, "groups": {"count": 4, "keep": 2}, "identity": 0, "top": top}, "shared": {"ff": glu(sff)}}
+    meg_dense = {"ff": dff, "kind": "dense", "limit": 7.0}
+    meg = lambda mlps: DecoderLMConfig.from_dict({"architecture": "Megolorn", "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "vocab": V, "width": W,
+                                                  "layers": [{"type": "attention", "mixer": meg_mix, "mlp": m} for m in mlps]})
+    dib = lambda t, m: DecoderLMConfig.from_dict({"architecture": "Dibulix", "logit_scale": 0.5, "norm": {"eps": 1e-6}, "vocab": V, "width": W, "layers": [{"type": t, "mixer": m, "mlp": None}] * 2})
+    mlps = [moe if k == "attention" else dense for k in kinds]
+    whole = list(zip(kinds, mlps))
+    return {"korirax": kor(whole, side), "korirax_looped": kor(whole, side, (1, len(kinds), 2)),
+            "megolorn_equal": meg([meg_moe if k == "attention" else meg_dense for k in kinds]),
+            "korirax/latent_attention": kor([("latent_attention", None)] * 2),
+            "dibulix/latent_attention": dib("latent_attention", {"dim": d, "heads": H, "kv_rank": r, "rot_dim": rd, "rot": {"base": 1e5, "dims": rd, "scaling": ramp}, "scale": (d + rd) ** -0.5, "vdim": d}),
+            "korirax/attention": kor([("attention", None)] * 2), "megolorn/attention": meg([None] * 2),
+            "korirax/rglru": kor([("rglru", None)] * 2),
+            "dibulix/mingru": dib("parallel", {"left": {"dim": 16, "heads": 1, "kv_heads": 1, "mask": {"size": 16}, "scale": 0.25, "vdim": 16}, "left_scale": 1.0,
+                                               "right": {"width": N}, "right_scale": 1.0}),
+            "korirax/dense": kor([("attention", dense)] * 2), "megolorn/dense": meg([meg_dense] * 2),
+            "korirax/moe": kor([("attention", moe)] * 2), "megolorn/moe": meg([meg_moe] * 2),
+            "korirax/token_input": kor([("attention", None)] * 2, side)}
+
+
+def korirax_arm(args) -> None:
+    """Prefill (one prompt of --prefill-tokens) and decode (--decode-batch requests, one token each, on --context cached tokens)
+    of the Korirax design with random weights, per size: whole steps, and per class of kernel for small models of one mechanism,
+    each beside the like kernel of the existing design that has it, against the measured rooflines."""
+    from moshi_b200 import _lib
+    from moshi_b200.models import DecoderLM, DecoderLMGen
+    from moshi_b200.synth import iter_synth_decoder_tensors
+    device = torch.device("cuda:0")
+    torch.cuda.set_device(device)
+    hbm, src = _peaks()
+    pk = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
+    tf = float(pk.get("bf16_tflops", 1590.0))
+    T, B, ctx = args.prefill_tokens, args.decode_batch, args.context
+    g = torch.Generator().manual_seed(7)
+    out = {"impl": "b200", "mode": "decoder-lm", "arch": "korirax", "dtype": "bf16", "data": "synthetic (random weights)",
+           "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src}, "workload": {"prefill_tokens": T, "decode_batch": B, "context": ctx}, "sizes": {}}
+    launches0 = _lib.lib().b200_launch_count()
+
+    def measure(cfg):
+        # random corrections would send every token to the same few experts: none, so that the experts' load is even
+        tensors = ((k, torch.zeros_like(t) if k.endswith("correction") else t) for k, t in iter_synth_decoder_tensors(cfg, seed=11, device=device))
+        model = DecoderLM(cfg, tensors, device=device)
+        gen = DecoderLMGen(model, slots=B, capacity=ctx + 64, max_step_tokens=max(T, B), max_want=B)
+        V = cfg.vocab
+        prompt = torch.randint(0, V, (T,), generator=g).tolist()
+
+        def prefill():
+            gen.step([(0, prompt)], [T - 1])
+            gen.release(0)
+
+        def classes(fn):
+            gen.set_option("time_kernels", 1)
+            gen.kernel_times()
+            for _ in range(3):
+                fn()
+            kt = {k: v / 3 for k, v in gen.kernel_times().items()}
+            gen.set_option("time_kernels", 0)
+            return kt
+        res = {"prefill": {"ms": _timed_steps(prefill, args.steps, args.warmup)}}
+        fl = model.algorithmic_flops(T, 0)
+        res["prefill"].update({"tokens_per_s": T / res["prefill"]["ms"] * 1e3, "kernel_ms": classes(prefill), "tflops": fl / res["prefill"]["ms"] / 1e9,
+                               "frac_of_bf16_peak": fl / res["prefill"]["ms"] / 1e9 / tf})
+        filler = torch.randint(0, V, (ctx,), generator=g).tolist()
+        for b in range(B):
+            for a in range(0, ctx, max(T, B)):
+                gen.step([(b, filler[a:a + max(T, B)])], [])
+        toks = torch.randint(0, V, (B,), generator=g).tolist()
+
+        def decode():
+            gen.step([(b, [toks[b]]) for b in range(B)], list(range(B)))
+        res["decode"] = {"ms": _timed_steps(decode, min(args.steps, 40), min(args.warmup, 5))}
+        nbytes = model.algorithmic_bytes(B, B * ctx)
+        res["decode"].update({"tokens_per_s": B / res["decode"]["ms"] * 1e3, "kernel_ms": classes(decode), "algorithmic_bytes": nbytes,
+                              "frac_of_hbm_peak": nbytes / res["decode"]["ms"] / 1e6 / hbm})
+        assert gen.error_flags() == 0
+        gen.close()
+        del gen, model
+        torch.cuda.empty_cache()
+        return res
+
+    for size in args.decoder_sizes.split(","):
+        W, kinds, H, G, d, rd, r, qr, N, nb, E, top, ff, sff, dff, side, V = KORIRAX_SIZES[size]
+        res = {"config": dict(zip(("width", "layers", "heads", "kv_heads", "head_dim", "rot_dim", "kv_rank", "q_rank", "recurrence_width", "blocks", "experts", "top", "expert_ff",
+                                   "shared_ff", "dense_ff", "token_input", "vocab"), KORIRAX_SIZES[size])), "models": {}}
+        for name, cfg in _korirax_cfgs(size).items():
+            res["models"][name] = measure(cfg)
+        m = res["models"]
+        pc, rp, glu = T * (T + 1) // 2, (r + rd + 63) // 64 * 64, ff * 2 // 3 // 64 * 64
+
+        def per_layer(name, phase, cls):
+            return m[name][phase]["kernel_ms"][cls] / 2
+
+        def tflops(name, cls, fl):
+            return fl / per_layer(name, "prefill", cls) / 1e9 / tf
+
+        def hbm_frac(name, phase, cls, nbytes):
+            return nbytes / per_layer(name, phase, cls) / 1e6 / hbm
+        # fractions of the measured peaks of one layer's kernels: tensor-core FLOPs in prefill, bytes in decode (state and element-wise ones: bytes in both)
+        used = min(E, B * top)
+        lat_fl, lat_b, att_b = 4 * pc * H * (r + rd), B * (ctx + 1) * rp * 2, B * (ctx + 1) * 2 * G * d * 2
+        lin_k, lin_m = (2 * H + 2 * G) * d * W + H * d * W + 3 * dff * W, (H + 2 * G) * d * W + H * d * W + 3 * dff * W      # q, k, v, (gate), o, the gated unit
+        # RG-LRU: x and y read (bf16), u written and read (fp32), coefficients written and read twice, result written; minGRU: z, x, g read, result written
+        rg_rec, rg_gate_w = T * N * (4 + 8 + 8 + 2 + 2), 2 * N * (N // nb) * 2
+        res["like_kernels"] = {
+            "latent_attention": {"prefill_frac_of_bf16_peak": {"korirax": tflops("korirax/latent_attention", "attention", lat_fl), "dibulix": tflops("dibulix/latent_attention", "attention", lat_fl)},
+                                 "decode_frac_of_hbm_peak": {"korirax": hbm_frac("korirax/latent_attention", "decode", "attention", lat_b),
+                                                             "dibulix": hbm_frac("dibulix/latent_attention", "decode", "attention", lat_b)}},
+            "attention": {"prefill_frac_of_bf16_peak": {"korirax": tflops("korirax/attention", "attention", 4 * pc * H * d), "megolorn": tflops("megolorn/attention", "attention", 2 * pc * H * 3 * d)},
+                          "decode_frac_of_hbm_peak": {"korirax": hbm_frac("korirax/attention", "decode", "attention", att_b), "megolorn": hbm_frac("megolorn/attention", "decode", "attention", att_b)}},
+            "recurrence": {"prefill_frac_of_hbm_peak": {"korirax": hbm_frac("korirax/rglru", "prefill", "recurrent", rg_rec), "dibulix_mingru": hbm_frac("dibulix/mingru", "prefill", "recurrent", T * N * 8)},
+                           "prefill_ms_per_layer": {"korirax": per_layer("korirax/rglru", "prefill", "recurrent"), "dibulix_mingru": per_layer("dibulix/mingru", "prefill", "recurrent")},
+                           "decode_frac_of_hbm_peak": {"korirax": hbm_frac("korirax/rglru", "decode", "recurrent", rg_gate_w + B * N * (4 + 4 + 4 + 2 + 2)),
+                                                       "dibulix_mingru": hbm_frac("dibulix/mingru", "decode", "recurrent", B * N * (8 + 8))},
+                           "decode_ms_per_layer": {"korirax": per_layer("korirax/rglru", "decode", "recurrent"), "dibulix_mingru": per_layer("dibulix/mingru", "decode", "recurrent")}},
+            "linear": {"prefill_frac_of_bf16_peak": {"korirax": tflops("korirax/dense", "linear", 2 * T * lin_k), "megolorn": tflops("megolorn/dense", "linear", 2 * T * lin_m)},
+                       "decode_frac_of_hbm_peak": {"korirax": hbm_frac("korirax/dense", "decode", "linear", lin_k * 2 + V * W), "megolorn": hbm_frac("megolorn/dense", "decode", "linear", lin_m * 2 + V * W)}},
+            "experts": {"prefill_frac_of_bf16_peak": {"korirax": tflops("korirax/moe", "experts", 4 * T * top * W * ff), "megolorn": tflops("megolorn/moe", "experts", 6 * T * top * W * glu)},
+                        "decode_frac_of_hbm_peak": {"korirax": hbm_frac("korirax/moe", "decode", "experts", used * 2 * ff * W * 2), "megolorn": hbm_frac("megolorn/moe", "decode", "experts", used * 3 * glu * W * 2)}},
+            "elementwise_ms_per_layer": {k: {ph: per_layer(k, ph, "elementwise") for ph in ("prefill", "decode")} for k in
+                                         ("korirax/latent_attention", "dibulix/latent_attention", "korirax/attention", "megolorn/attention", "korirax/rglru", "dibulix/mingru", "korirax/dense", "megolorn/dense")},
+            "fold_ms_per_layer": {k: {ph: per_layer(k, ph, "fold") for ph in ("prefill", "decode")} for k in
+                                  ("korirax/latent_attention", "dibulix/latent_attention", "korirax/moe", "megolorn/moe")},
+            "token_input_ms_per_layer": {ph: {c: per_layer("korirax/token_input", ph, c) - per_layer("korirax/attention", ph, c) for c in ("fold", "elementwise")} for ph in ("prefill", "decode")}}
+        out["sizes"][size] = res
+    out["gpu_launches"] = int(_lib.lib().b200_launch_count() - launches0)
+    print(json.dumps(out))
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1185,18 +1347,19 @@ def main() -> None:
     ap.add_argument("--decoder-lm", action="store_true",
                     help="instead of the default workload: prefill / decode throughput of the text-only decoder LM (Likosun design, random "
                          "weights) beside the Moshi temporal transformer at equal width and depth; prints its own JSON line")
-    ap.add_argument("--decoder-arch", choices=["likosun", "govuvik", "namalix", "dibulix", "megolorn"], default="likosun",
+    ap.add_argument("--decoder-arch", choices=["likosun", "govuvik", "namalix", "dibulix", "megolorn", "korirax"], default="likosun",
                     help="with --decoder-lm: which design to time (govuvik: window attention beside gated linear attention, mLSTM, routed experts; "
                          "namalix: sigmoid attention, retention, delta rule, clamped routed experts; dibulix: residual streams, latent attention "
                          "with a rotated key part, window attention beside a minGRU, delta rule with a decay per key channel; megolorn: differential attention "
-                         "on chunks, softmax-routed experts with groups and a shared expert)")
+                         "on chunks, softmax-routed experts with groups and a shared expert; korirax: latent attention with a query latent, attention with a distance bias, RG-LRU, "
+                         "sigmoid-routed erf-GELU experts, a per-layer token input)")
     ap.add_argument("--decoder-sizes", default="w2048,w4096", help="comma-separated names out of " + ",".join(DECODER_SIZES))
     ap.add_argument("--prefill-tokens", type=int, default=2048)
     ap.add_argument("--decode-batch", type=int, default=32)
     ap.add_argument("--context", type=int, default=2048)
     args = ap.parse_args()
     if args.decoder_lm:
-        {"govuvik": govuvik_arm, "namalix": namalix_arm, "dibulix": dibulix_arm, "megolorn": megolorn_arm}.get(args.decoder_arch, decoder_lm_arm)(args)
+        {"govuvik": govuvik_arm, "namalix": namalix_arm, "dibulix": dibulix_arm, "megolorn": megolorn_arm, "korirax": korirax_arm}.get(args.decoder_arch, decoder_lm_arm)(args)
         return
     if args.impl == "reference":
         reference_arm(args)

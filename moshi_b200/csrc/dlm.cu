@@ -83,8 +83,8 @@ struct Layer {
   float lambda = 0.f;
   // ---- joint layers of the parallel-residual block (finalize_joint_layer): as above one projection and one output product.  Latent
   // attention [dq | dkv | g | ..] with the queries' second product `uq`; bias attention [q | k | v | g | ..]; RG-LRU [y | x | ..]
-  Weight uq, side_gate, side_proj;
-  void* side_gate_rm = nullptr;        // T [side_dim][width], row-major (the few-token kernel)
+  Weight uq, side_proj;                // side_proj keeps its row-major form beside the packed one
+  void *side_gate = nullptr;           // T [side_dim][width]
   float *side_norm = nullptr, *rel = nullptr;      // rel: [heads][far + 1] biases over distances
   int far = 0, far_smem = 0;
   float *conv_b = nullptr, *x_b = nullptr, *y_b = nullptr, *gate_b = nullptr, *lam8 = nullptr;
@@ -1377,12 +1377,7 @@ int finalize_joint_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
   B200_TRY(put_joint_output(h, L, m + "o", unit + "down", Kv, drop));
   if (c.side_dim > 0) {
     const int D = c.side_dim;
-    B200_TRY(matrix(p + "side.gate", D, W, &L.side_gate_rm));
-    L.side_gate.rm = L.side_gate_rm; L.side_gate.N = D; L.side_gate.K = (int)W;      // kept row-major as well: the few-token kernel reads it
-    if (!h->f32 && h->use_tc && W % 8 == 0 && (D + 127) / 128 <= tc::SK_MAX_TILES) {
-      B200_TRY(h->weights.alloc(&L.side_gate.tiles, tc::sk_packed_bytes(D, (int)W, 0, 0), false));
-      B200_TRY(tc::sk_pack_weights(static_cast<const bf16*>(L.side_gate_rm), L.side_gate.tiles, D, (int)W, 0, 0, nullptr));
-    }
+    B200_TRY(matrix(p + "side.gate", D, W, &L.side_gate));
     void *proj = nullptr, *tmp = nullptr;
     B200_TRY(h->weights.alloc(&proj, (size_t)W * h->side_ld * es, true));
     B200_CUDA(cudaMalloc(&tmp, (size_t)W * D * es));
@@ -1391,7 +1386,9 @@ int finalize_joint_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
     cudaDeviceSynchronize();
     cudaFree(tmp);
     B200_TRY(rc);
-    B200_TRY(seal_weight(h, L.side_proj, proj, (int)W, h->side_ld, drop, (int)W));
+    std::vector<void*> keep;               // the row-major form stays: prompts read it
+    B200_TRY(seal_weight(h, L.side_proj, proj, (int)W, h->side_ld, keep, (int)W));
+    L.side_proj.rm = proj;
     B200_TRY(get_f32(h, p + "side.norm", W, &L.side_norm));
   }
   return B200_OK;
@@ -1757,19 +1754,23 @@ int token_input(b200_dlm* h, const Layer& L, int n_tok, float* trace, const floa
   const int W = h->cfg.width, D = h->cfg.side_dim, off = L.index * D;
   cudaStream_t st = h->stream;
   const int* tok = h->meta_dev + h->off_tok;
-  T *z = static_cast<T*>(h->sidez), *hb = static_cast<T*>(h->hbuf), *y = static_cast<T*>(h->mixo);
+  T *z = static_cast<T*>(h->sidez), *y = static_cast<T*>(h->mixo);
   const T* table = static_cast<const T*>(h->side_embed);
   if (n_tok <= SIDE_FEW) {
-    TIMED(CLS_FOLD, B200_LAUNCH(side_gate_kernel<T>, dim3(n_tok, ceil_div(D, 8)), 256, 0, st, h->xin, W, static_cast<const T*>(L.side_gate_rm), table, (long long)h->side_cols, off, tok,
-                                h->cfg.vocab, D, z, (long long)h->side_ld, W % 8 == 0));
+    TIMED(CLS_FOLD, B200_LAUNCH(side_gate_kernel<T>, dim3(n_tok, ceil_div(D, 8)), 256, 0, st, h->xin, W, static_cast<const T*>(L.side_gate), table, (long long)h->side_cols, off, tok,
+                                h->cfg.vocab, D, z, (long long)h->side_ld, W % 8 == 0);
+          B200_TRY(linear<T>(h, z, (long long)h->side_ld, L.side_proj, y, W, n_tok)));
   } else {
-    TIMED(CLS_FOLD, B200_TRY(linear<T>(h, hb, W, L.side_gate, z, h->side_ld, n_tok));
+    // both products are small in one direction: they run whole on 64 x 64 tiles, where the linears' kernel takes 256 rows at a time
+    TIMED(CLS_FOLD, B200_TRY(head_gemm(st, static_cast<const float*>(h->xin), (long long)W, 0, static_cast<const T*>(L.side_gate), (long long)W, 0, z, (long long)h->side_ld, 0,
+                                       n_tok, D, W, 1, 1.f, h->attn_tc != 0));
           B200_LAUNCH(side_act_kernel<T>, (unsigned)ceil_div64((int64_t)n_tok * D, 256), 256, 0, st, z, (long long)h->side_ld, table, (long long)h->side_cols, off, tok, h->cfg.vocab, D,
-                      (long long)n_tok * D));
+                      (long long)n_tok * D);
+          B200_TRY(head_gemm(st, static_cast<const T*>(z), (long long)h->side_ld, 0, static_cast<const T*>(L.side_proj.rm), (long long)h->side_ld, 0, y, (long long)W, 0,
+                             n_tok, W, h->side_ld, 1, 1.f, h->attn_tc != 0)));
   }
-  TIMED(CLS_FOLD, B200_TRY(linear<T>(h, z, (long long)h->side_ld, L.side_proj, y, W, n_tok)));
   auto end = n_tok <= 592 && W <= 4096 ? side_end_kernel<T, true> : side_end_kernel<T, false>;
-  TIMED(CLS_ELEMENTWISE, B200_LAUNCH(end, n_tok, 256, 0, st, h->xin, y, L.side_norm, trace, step, w_next, hb, W, h->cfg.norm_eps));
+  TIMED(CLS_ELEMENTWISE, B200_LAUNCH(end, n_tok, 256, 0, st, h->xin, y, L.side_norm, trace, step, w_next, static_cast<T*>(h->hbuf), W, h->cfg.norm_eps));
   return check_launch("token_input");
 }
 
@@ -1970,12 +1971,12 @@ int step_parallel(b200_dlm* h, int n_tok, int n_want, int max_ctx, float* logits
       TIMED(CLS_EXPERTS, B200_TRY(routed_experts_glu<T>(h, L, hb, n_tok)));
       yexp = static_cast<const T*>(h->yexp);
     }
-    const bool side = c.side_dim > 0, copy = side && n_tok > SIDE_FEW;      // the token input comes behind the sum: it reads the residual, or its rounding for many tokens
-    auto block_end = n_tok <= 592 && W <= 4096 && !copy ? parallel_block_end_kernel<T, true> : parallel_block_end_kernel<T, false>;
+    const bool side = c.side_dim > 0;      // the token input comes behind the sum
+    auto block_end = n_tok <= 592 && W <= 4096 ? parallel_block_end_kernel<T, true> : parallel_block_end_kernel<T, false>;
     float* trace = h->trace_layers ? h->trace + (long long)li * stride : nullptr;
     const float *step = last ? nullptr : h->layers[li + 1].step, *w_next = last ? nullptr : h->layers[li + 1].n1w;
     TIMED(CLS_ELEMENTWISE, B200_LAUNCH(block_end, n_tok, 256, 0, st, h->xin, mixo, ffo, yexp, h->moe_w, L.c.top, side ? nullptr : trace, side ? nullptr : w_next, hb, W, c.norm_eps,
-                                       copy ? ROW_COPY : c.norm == B200_NORM_LAYER ? ROW_LAYER : ROW_RMS,
+                                       c.norm == B200_NORM_LAYER,
                                        L.c.identity > 0 ? h->moe_idx : (const int*)nullptr, L.c.experts, side ? nullptr : step));
     if (side) B200_TRY(token_input<T>(h, L, n_tok, trace, step, w_next));
   }
@@ -2513,7 +2514,7 @@ int b200_dlm_finalize(b200_dlm* h) {
   if (parallel) {
     h->vmix_first = -1;
     if (c.side_dim > 0) {
-      h->side_ld = (c.side_dim + 7) / 8 * 8; h->side_cols = c.n_layers * c.side_dim;
+      h->side_ld = (c.side_dim + 15) / 16 * 16; h->side_cols = c.n_layers * c.side_dim;
       B200_TRY(matrix("side.embed", c.vocab, h->side_cols, &h->side_embed));      // gathered, like the embedding
     }
     for (int i = 0; i < c.n_layers; ++i) {

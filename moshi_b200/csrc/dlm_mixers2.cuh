@@ -21,15 +21,10 @@ __device__ __forceinline__ float clamped_gluf(float g, float u, float limit) {
   return g * sigmoidf(1.702f * g) * (u + 1.f);
 }
 
-// the block's norm of one fp32 row -> T (`layer`): ROW_RMS (w as it is multiplied), ROW_LAYER without a bias, ROW_COPY: the row itself
-enum { ROW_RMS = 0, ROW_LAYER = 1, ROW_COPY = 2 };
+// the block's norm of one fp32 row -> T: layer norm without a bias, or RMS norm (w as it is multiplied)
 template <typename T>
 __device__ __forceinline__ void block_norm(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ h, int W, float eps, int layer, float* red) {
-  if (layer == ROW_COPY) {
-    for (int i = threadIdx.x; i < W; i += blockDim.x) h[i] = from_f<T>(x[i]);
-    return;
-  }
-  if (layer == ROW_LAYER) { block_layernorm<T>(x, w, nullptr, h, W, eps, red); return; }
+  if (layer) { block_layernorm<T>(x, w, nullptr, h, W, eps, red); return; }
   const float r = block_rrms(x, W, eps, red);
   for (int i = threadIdx.x; i < W; i += blockDim.x) h[i] = from_f<T>(x[i] * r * w[i]);
 }
@@ -53,8 +48,7 @@ __global__ void __launch_bounds__(256) embed_scale_norm_kernel(const int* __rest
 
 // End of a parallel block, one CTA per token:  x <- x + mix + ff,  ff = a dense feed-forward's row | sum_k ew[t][k] * rows of
 // the chosen experts (the row of h itself for a choice from n_exp on: an identity expert) | both | nothing;  optional copy of x
-// (per-layer trace);  x <- x + step (the vector in front of a pass, when given);  optional h = norm(x) * w_next for the next layer
-// (layer = ROW_COPY, not with REG: h = x as it is).
+// (per-layer trace);  x <- x + step (the vector in front of a pass, when given);  optional h = norm(x) * w_next for the next layer.
 // REG (few tokens, W <= 4096): the row stays in registers between the sum and the norm, which shortens the chain of a CTA; many tokens
 // fill the SMs better with the smaller kernel.
 template <typename T, bool REG>
@@ -116,7 +110,7 @@ __global__ void __launch_bounds__(256) parallel_block_end_kernel(float* __restri
     if (step) v += step[i];
     x[i] = v;
   }
-  if (w_next || layer == ROW_COPY) {
+  if (w_next) {
     __syncthreads();
     block_norm<T>(x, w_next, h + t * W, W, eps, layer, red);
   }

@@ -165,7 +165,7 @@ def test_mechanisms_in_isolation(what, side):
 
 
 @BOTH
-@pytest.mark.parametrize("buckets,far", [(32, 100), (8, 40), (6, 64), (20, 131), (2, 3), (12, 7)])
+@pytest.mark.parametrize("buckets,far", [(32, 100), (8, 40), (6, 64), (20, 131), (4, 5), (12, 7)])
 def test_bias_buckets_at_their_edges(buckets, far, dtype):
     """Large table entries of alternating sign, so that a distance in the wrong bucket shows; the oracle itself moves by far more than
     the tolerance when an edge moves by one.  bfloat16 takes the tensor-core kernels, with the table in shared memory."""
@@ -181,7 +181,7 @@ def test_bias_buckets_at_their_edges(buckets, far, dtype):
     toks = tokens(n, cfg.vocab, 3)
     want = orc.forward(toks)
     moved = cfg.to_dict()
-    moved["layers"][0]["mixer"]["bias_max"] = far * 1.15 + 1
+    moved["layers"][0]["mixer"]["bias_max"] = far * 1.5 + 1
     moves(Oracle(moved, orc.t).forward(toks), want, dtype, 20 if dtype == torch.float32 else 1.5)
     with gen_for(model, capacity=n + 8, max_step_tokens=max(256, n)) as gen:
         def close(got, what):
@@ -336,7 +336,7 @@ def test_loops_anywhere_with_a_cache_per_pass(loop):
             assert_close(in_portions(gen, 1, toks, [31, 2, 5] + [1] * 20), want, torch.float32, "portions")
 
 
-@pytest.mark.parametrize("side", [1, 8, 24, 100])
+@pytest.mark.parametrize("side", [3, 8, 24, 100])
 def test_token_input_for_few_and_many_tokens(side):
     """Up to 64 tokens take the one-launch gate product, more the GEMM: both, in both precisions; the oracle moves when the layers'
     parts of the second table are exchanged."""
