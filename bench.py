@@ -1261,7 +1261,7 @@ def korirax_arm(args) -> None:
             gen.set_option("time_kernels", 0)
             return kt
         res = {"prefill": {"ms": _timed_steps(prefill, args.steps, args.warmup)}}
-        fl = model.algorithmic_flops(T, 0)
+        fl = model.algorithmic_flops(T, 0) - 2 * (T - 1) * cfg.width * V      # logits of the last token only
         res["prefill"].update({"tokens_per_s": T / res["prefill"]["ms"] * 1e3, "kernel_ms": classes(prefill), "tflops": fl / res["prefill"]["ms"] / 1e9,
                                "frac_of_bf16_peak": fl / res["prefill"]["ms"] / 1e9 / tf})
         filler = torch.randint(0, V, (ctx,), generator=g).tolist()

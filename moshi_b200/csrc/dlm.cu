@@ -1330,7 +1330,10 @@ int finalize_joint_layer(b200_dlm* h, int i, std::vector<void*>& drop) {
     const int n = a.dim, nb = a.blocks, bs = n / nb;
     B200_TRY(get_f32(h, m + "x.b", n, &L.x_b));
     B200_TRY(get_f32(h, m + "y.b", n, &L.y_b));
-    B200_TRY(get_f32_shaped(h, m + "conv", {n, a.conv_taps}, &L.qkv_conv));
+    float* conv = nullptr;               // [channels][taps] -> [taps][channels]
+    B200_TRY(get_f32_shaped(h, m + "conv", {n, a.conv_taps}, &conv));
+    B200_TRY(h->weights.alloc_t(&L.qkv_conv, (size_t)n * a.conv_taps, false));
+    B200_LAUNCH(head_transpose_kernel<float>, (unsigned)ceil_div64((int64_t)n * a.conv_taps, 256), 256, 0, nullptr, conv, L.qkv_conv, 1, n, a.conv_taps);
     B200_TRY(get_f32(h, m + "conv.b", n, &L.conv_b));
     float *lam = nullptr, *rb = nullptr, *ib = nullptr;
     B200_TRY(get_f32(h, m + "lam", n, &lam));

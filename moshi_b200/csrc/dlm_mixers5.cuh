@@ -79,7 +79,7 @@ __global__ void __launch_bounds__(128) latent_query_rope_kernel(const T* __restr
 struct RgLruParams {
   const void* proj; long long ld;       // T [tokens][ld]
   int off_x, off_y, C, taps, bs;        // bs = channels of a gate matrix
-  const float *bx, *by, *conv, *bc;     // conv [C][taps]
+  const float *bx, *by, *conv, *bc;     // conv [taps][C]
   float* hist;                          // [slots][taps - 1][C]
   float* u;                             // [tokens][C]
   const void* gates;                    // T [C / bs][2 bs][bs], rows 2c / 2c + 1 = r / i of the block's channel c
@@ -111,11 +111,16 @@ __global__ void __launch_bounds__(256) rglru_conv_kernel(RgLruParams p) {
   float* hist = p.hist + (long long)p.tok_slot[t] * keep * p.C;
   for (int c = blockIdx.y * CONV_SLICE + threadIdx.x; c < c1; c += 256) {
     const float b = p.bx[c], own = to_f(row[p.off_x + c]) + b;
-    const float* w = p.conv + (long long)c * p.taps;
-    float acc = fmaf(w[keep], own, p.bc[c]);
-    for (int k = 1; k <= keep && k <= pos; ++k) {
-      const float v = k <= back ? to_f(row[p.off_x + c - k * p.ld]) + b : hist[(long long)((pos - k) % keep) * p.C + c];
-      acc = fmaf(w[keep - k], v, acc);
+    const float* w = p.conv + c;
+    float acc = fmaf(w[(long long)keep * p.C], own, p.bc[c]);
+    if (back >= keep) {        // every tap lies inside the step
+#pragma unroll 4
+      for (int k = 1; k <= keep; ++k) acc = fmaf(w[(long long)(keep - k) * p.C], to_f(row[p.off_x + c - k * p.ld]) + b, acc);
+    } else {
+      for (int k = 1; k <= keep && k <= pos; ++k) {
+        const float v = k <= back ? to_f(row[p.off_x + c - k * p.ld]) + b : hist[(long long)((pos - k) % keep) * p.C + c];
+        acc = fmaf(w[(long long)(keep - k) * p.C], v, acc);
+      }
     }
     p.u[t * p.C + c] = acc;
     if (only && keep > 0) hist[(long long)(pos % keep) * p.C + c] = own;
