@@ -1726,7 +1726,9 @@ int rglru(b200_dlm* h, const Layer& L, int n_tok) {
   p.tok_slot = meta + h->off_slot; p.tok_pos = meta + h->off_pos; p.tok_first = meta + h->off_first; p.tok_last = meta + h->off_last;
   p.ent_tok0 = meta + h->off_whole_tok0; p.ent_ntok = meta + h->off_whole_ntok; p.ent_slot = meta + h->off_whole_slot; p.ent_pos0 = meta + h->off_whole_pos0;
   p.n_tok = n_tok; p.unit = unit_params<T>(h, L); p.conv_rows = ceil_div(p.C, CONV_SLICE);
-  TIMED(CLS_ELEMENTWISE, B200_LAUNCH(rglru_conv_kernel<T>, dim3(n_tok, p.conv_rows + ceil_div(L.glu_ff, GLU_SLICE)), 256, 0, st, p);
+  const int conv_grid = p.conv_rows + ceil_div(L.glu_ff, GLU_SLICE);
+  TIMED(CLS_ELEMENTWISE, if (n_tok >= 512) B200_LAUNCH((rglru_conv_kernel<T, 8>), dim3(ceil_div(n_tok, 8), conv_grid), 256, 0, st, p);
+        else B200_LAUNCH((rglru_conv_kernel<T, 1>), dim3(n_tok, conv_grid), 256, 0, st, p);
         if (p.taps > 1 && h->max_entry_tokens > 1)
           B200_LAUNCH(conv_carry_kernel<T>, n_tok, 256, 0, st, static_cast<const T*>(h->proj) + L.g_x, (long long)L.ldp, L.qkv_hist, p.C, p.taps - 1, p.tok_slot, p.tok_pos,
                       p.tok_last, L.x_b));

@@ -96,34 +96,52 @@ struct RgLruParams {
 
 constexpr int CONV_SLICE = 512;
 
-// grid (tokens, conv_rows + slices): u on CONV_SLICE channels each; then the feed-forward's unit.  A token that is its request's only one
-// in the step also puts its input into the carried rows (it alone reads them); conv_carry_kernel does so for longer portions.
-template <typename T>
+// grid (tokens / TT, conv_rows + slices): u on CONV_SLICE channels of TT neighbouring tokens each (many tokens: their loads overlap and
+// share the taps); then the feed-forward's unit.  A token that is its request's only one in the step also puts its input into the
+// carried rows (it alone reads them); conv_carry_kernel does so for longer portions.
+template <typename T, int TT>
 __global__ void __launch_bounds__(256) rglru_conv_kernel(RgLruParams p) {
-  const long long t = blockIdx.x;
-  const T* row = static_cast<const T*>(p.proj) + t * p.ld;
+  const long long t0 = (long long)blockIdx.x * TT;
+  const int nt = TT == 1 ? 1 : (int)min((long long)TT, p.n_tok - t0);
+  const T* row0 = static_cast<const T*>(p.proj) + t0 * p.ld;
   if ((int)blockIdx.y >= p.conv_rows) {
-    unit_slice<T>(p.unit, row, p.ld, t, ((int)blockIdx.y - p.conv_rows) * GLU_SLICE);
+    for (int j = 0; j < nt; ++j) unit_slice<T>(p.unit, row0 + j * p.ld, p.ld, t0 + j, ((int)blockIdx.y - p.conv_rows) * GLU_SLICE);
     return;
   }
-  const int pos = p.tok_pos[t], back = (int)t - p.tok_first[t], keep = p.taps - 1, c1 = min(p.C, ((int)blockIdx.y + 1) * CONV_SLICE);
-  const bool only = p.tok_first[t] == p.tok_last[t];
-  float* hist = p.hist + (long long)p.tok_slot[t] * keep * p.C;
+  const int keep = p.taps - 1, c1 = min(p.C, ((int)blockIdx.y + 1) * CONV_SLICE);
+  // every tap of every token of the tile lies inside the step
+  const bool inside = nt == TT && (int)t0 - p.tok_first[t0] >= keep && p.tok_last[t0] >= (int)t0 + TT - 1;
   for (int c = blockIdx.y * CONV_SLICE + threadIdx.x; c < c1; c += 256) {
-    const float b = p.bx[c], own = to_f(row[p.off_x + c]) + b;
+    const float b = p.bx[c], bc = p.bc[c];
     const float* w = p.conv + c;
-    float acc = fmaf(w[(long long)keep * p.C], own, p.bc[c]);
-    if (back >= keep) {        // every tap lies inside the step
-#pragma unroll 4
-      for (int k = 1; k <= keep; ++k) acc = fmaf(w[(long long)(keep - k) * p.C], to_f(row[p.off_x + c - k * p.ld]) + b, acc);
-    } else {
+    const T* x = row0 + p.off_x + c;
+    if (TT > 1 && inside) {
+      float acc[TT];
+      const float wk = w[(long long)keep * p.C];
+#pragma unroll
+      for (int j = 0; j < TT; ++j) acc[j] = fmaf(wk, to_f(x[j * p.ld]) + b, bc);
+      for (int k = 1; k <= keep; ++k) {
+        const float wv = w[(long long)(keep - k) * p.C];
+#pragma unroll
+        for (int j = 0; j < TT; ++j) acc[j] = fmaf(wv, to_f(x[(j - k) * p.ld]) + b, acc[j]);
+      }
+#pragma unroll
+      for (int j = 0; j < TT; ++j) p.u[(t0 + j) * p.C + c] = acc[j];
+      continue;
+    }
+    for (int j = 0; j < nt; ++j) {
+      const long long t = t0 + j;
+      const int pos = p.tok_pos[t], back = (int)t - p.tok_first[t];
+      float* hist = p.hist + (long long)p.tok_slot[t] * keep * p.C;
+      const float own = to_f(x[j * p.ld]) + b;
+      float acc = fmaf(w[(long long)keep * p.C], own, bc);
       for (int k = 1; k <= keep && k <= pos; ++k) {
-        const float v = k <= back ? to_f(row[p.off_x + c - k * p.ld]) + b : hist[(long long)((pos - k) % keep) * p.C + c];
+        const float v = k <= back ? to_f(x[(j - k) * p.ld]) + b : hist[(long long)((pos - k) % keep) * p.C + c];
         acc = fmaf(w[(long long)(keep - k) * p.C], v, acc);
       }
+      p.u[t * p.C + c] = acc;
+      if (keep > 0 && p.tok_first[t] == p.tok_last[t]) hist[(long long)(pos % keep) * p.C + c] = own;
     }
-    p.u[t * p.C + c] = acc;
-    if (only && keep > 0) hist[(long long)(pos % keep) * p.C + c] = own;
   }
 }
 

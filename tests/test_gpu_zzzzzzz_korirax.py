@@ -318,6 +318,23 @@ def test_recurrence_with_a_long_memory(width, blocks, conv, dtype):
             assert_close(got, wb[6:], dtype, "its next portion")
 
 
+@BOTH
+@pytest.mark.parametrize("conv", [1, 4, 7, 12])
+def test_convolution_in_steps_of_many_tokens(conv, dtype):
+    """Steps of at least 512 tokens take the convolution on tiles of eight tokens: one prompt, then requests of several lengths on
+    several histories whose borders cut the tiles, single tokens among them."""
+    cfg = make_cfg([rglru(36, 3, conv, mlp=dense(24)), rglru(32, 2, conv)], vocab=53, width=40, side=4)
+    model, orc = build(cfg, dtype, seed=19)
+    a, b, c, d = tokens(1060, cfg.vocab, 8), tokens(13, cfg.vocab, 9), tokens(4, cfg.vocab, 10), tokens(60, cfg.vocab, 11)
+    wa, wb, wc, wd = (orc.forward(x) for x in (a, b, c, d))
+    with gen_for(model, slots=4, capacity=1100, max_step_tokens=700) as gen:
+        assert_close(gen.step([(0, a[:519])], list(range(519))), wa[:519], dtype, "one prompt")
+        gen.step([(1, b[:12]), (3, d[:2])], [])
+        got = gen.step([(1, b[12:]), (3, d[2:]), (2, c), (0, a[519:])], list(range(1 + 58 + 4 + 541)))
+        for lo, w, what in ((0, wb[12:], "b"), (1, wd[2:], "d"), (59, wc, "c"), (63, wa[519:], "a")):
+            assert_close(got[lo:lo + len(w)], w, dtype, what)
+
+
 @pytest.mark.parametrize("loop", [(0, 1, 1), (0, 2, 2), (1, 2, 4), (0, 3, 2), (1, 3, 3), (2, 3, 2)])
 def test_loops_anywhere_with_a_cache_per_pass(loop):
     layers = [attention(2, 1, 8, 6, 0.4, far=20, buckets=8, mlp=dense(20)), rglru(18, 2, 3, mlp=moe(4, 2, 12)), latent(2, 6, 4, 5, 10, 8, 0.4)]
